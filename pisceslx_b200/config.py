@@ -58,6 +58,7 @@ class YvActivationType(str, Enum):
 class YvConfig:
     # ---- identity / sizes -------------------------------------------------------------------
     model_type: str = "piscesl1"
+    architecture: str = ""                  # name in ``architectures`` / ``models.registry``; "" = the Yv trunk
     vocab_size: int = 151646
     hidden_size: int = 2048
     n_layer: int = 24
@@ -219,6 +220,9 @@ class YvConfig:
     fp8_block_size: int = 128
     use_fp4: bool = False
     fp4_block_size: int = 16
+    # ---- layered architectures (``architectures`` fills these from a checkpoint's config.json) ----------------------
+    layer_specs: List[Dict[str, Any]] = field(default_factory=list)   # one {"mixer": ..., "mlp": ...} per layer
+    token_side_dim: int = 0                 # width of the per-layer token input (0 = none)
     # ---- task heads ---------------------------------------------------------------------------------------------
     task_classes: int = 256
     classifier_dropout: float = 0.1
@@ -274,6 +278,8 @@ class YvConfig:
     def validate(self) -> List[str]:
         """Return a list of problems (empty = valid); mirrors reference model/config.py:1267."""
         errs: List[str] = []
+        if self.layer_specs and len(self.layer_specs) != self.n_layer:
+            errs.append(f"{len(self.layer_specs)} layer specs for {self.n_layer} layers")
         if self.hidden_size <= 0 or self.n_layer <= 0:
             errs.append("hidden_size and n_layer must be positive")
         if self.n_head % self.n_kv_head != 0:
@@ -293,6 +299,8 @@ class YvConfig:
     # ---- parameter / memory estimates --------------------------------------------------------------------
     def count_parameters(self) -> Dict[str, int]:
         H = self.hidden_size
+        if self.layer_specs:
+            return self._count_layered()
         attn = H * self.q_dim + 2 * H * self.kv_dim + self.q_dim * H
         routed = self.moe_num_experts * 3 * H * self.moe_expert_intermediate_size
         shared = self.moe_shared_experts * 3 * H * self.moe_shared_intermediate_size
@@ -308,6 +316,22 @@ class YvConfig:
         active = n_moe * active_layer + n_dense * per_layer_dense + self.vocab_size * H
         return {"total": int(total), "active": int(active), "embedding": int(emb),
                 "per_layer": int(per_layer_moe if n_moe else per_layer_dense)}
+
+    def _count_layered(self) -> Dict[str, int]:
+        H, S = self.hidden_size, self.token_side_dim
+        total = 0
+        for spec in self.layer_specs:
+            m, f = spec["mixer"], spec["mlp"]
+            hd = m["heads"] * (m["dim"] + m["rot_dim"])
+            total += (H * (m["q_rank"] + m["kv_rank"] + m["rot_dim"] + (m["heads"] if m.get("output_gate") else 0))
+                      + hd * m["q_rank"] + m["heads"] * (m["dim"] + m["vdim"]) * m["kv_rank"] + H * m["heads"] * m["vdim"]
+                      + m["q_rank"] + m["kv_rank"] + 2 * H)
+            total += (2 * H * f["ff"] + 2 * H) if f else 0
+            total += (2 * H * S + H) if S else 0
+        emb = 2 * self.vocab_size * H
+        side = self.vocab_size * self.n_layer * S
+        return {"total": int(total + emb + side + 2 * H), "active": int(total + self.vocab_size * H),
+                "embedding": int(emb + side), "per_layer": int(total // max(self.n_layer, 1))}
 
     def estimate_memory_usage(self, batch: int = 1, seq: int = 4096, bytes_per_param: int = 2,
                               optimizer_bytes_per_param: int = 2, world: int = 1) -> Dict[str, float]:
@@ -332,6 +356,9 @@ class YvConfig:
     @classmethod
     def from_dict(cls, d: Dict[str, Any]) -> "YvConfig":
         d = dict(d or {})
+        if d.get("architecture") and not d.get("layer_specs"):
+            from .architectures import config_fields
+            return cls(**config_fields(d))
         names = {f.name for f in dataclasses.fields(cls)}
         known = {k: v for k, v in d.items() if k in names and k != "extra"}
         extra = dict(d.get("extra") or {})

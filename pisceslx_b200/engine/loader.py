@@ -3,7 +3,8 @@
 Follows the reference's loading contract: ``YvConfig.from_yaml(configs/model/<size>.yaml)`` -> model ->
 ``torch.load(ckpt)`` accepting ``model_state_dict | model | state_dict | raw`` (tools/infer/core.py:209-226,
 opss/infer/native_ruchbah.py:77-84); ``save_pretrained`` writes ``pytorch_model.bin`` + ``config.json``
-(model/core/model.py:1240-1253)."""
+(model/core/model.py:1240-1253).  A checkpoint may also be a folder with ``config.json`` naming an architecture and
+``model.safetensors`` (one file, or shards with an index): the folder then decides the model class and its sizes."""
 from __future__ import annotations
 
 import json
@@ -16,6 +17,7 @@ import torch
 from ..config import YvConfig
 from ..models import build_model
 from .checkpoint import extract_state_dict
+from .weights import read_folder
 
 REPO_ROOT = Path(__file__).resolve().parents[2]
 
@@ -50,18 +52,34 @@ def attach_optional_components(model: Any, cfg: YvConfig, parallel: Any = None) 
         attach_multimodal(model, vision=True)
 
 
+def folder_config(ckpt: Optional[str]) -> Optional[YvConfig]:
+    """Configuration of a checkpoint folder whose config.json names an architecture, else None."""
+    path = Path(ckpt) / "config.json" if ckpt else None
+    if path is None or not path.is_file():
+        return None
+    return YvConfig.from_json(path) if json.loads(path.read_text()).get("architecture") else None
+
+
+def _checkpoint_tensors(path: Path) -> Any:
+    if path.is_dir():
+        if (path / "pytorch_model.bin").exists():
+            path = path / "pytorch_model.bin"
+        else:
+            return read_folder(path)
+    return extract_state_dict(torch.load(path, map_location="cpu", weights_only=False))
+
+
 def load_model_for_inference(model_size: str = "0.01B", ckpt: Optional[str] = None, device: Optional[str] = None,
                              model_config: Optional[str] = None, dtype: Optional[torch.dtype] = None) -> Any:
-    cfg = resolve_model_config(model_size, model_config)
+    cfg = folder_config(ckpt) if model_config is None else None
+    named = cfg is not None
+    cfg = cfg or resolve_model_config(model_size, model_config)
     dev = torch.device(device) if device else torch.device("cuda" if torch.cuda.is_available() else "cpu")
     model = build_model(cfg, dev, dtype)
     attach_optional_components(model, cfg)
     if ckpt:
-        path = Path(ckpt)
-        if path.is_dir() and (path / "pytorch_model.bin").exists():
-            path = path / "pytorch_model.bin"
-        sd = extract_state_dict(torch.load(path, map_location="cpu", weights_only=False))
-        model.load_reference_state_dict(sd, strict=False)
+        # a folder that names its architecture is complete; the trunk's own checkpoints may lack optional parts
+        model.load_reference_state_dict(_checkpoint_tensors(Path(ckpt)), strict=named)
     return model.eval()
 
 

@@ -22,8 +22,9 @@ from __future__ import annotations
 
 import math
 from dataclasses import dataclass, field
-from typing import Any, Dict, Optional
+from typing import Any, Callable, Dict, List, Optional, Tuple
 
+import numpy as np
 import torch
 import torch.nn as nn
 
@@ -47,9 +48,32 @@ class AttnContext:
     block_table: Optional[torch.Tensor] = None   # int32 [B, max_blocks]
     seq_lens: Optional[torch.Tensor] = None      # int32 [B] lengths after this step
     decode: bool = False
+    max_position: int = 0                        # no position of the step is at or past this one (host value)
+    # a portion that continues cached sequences: tokens already cached and new tokens per sequence, and the flat cache
+    # slots of all of a sequence's tokens (host values)
+    starts: Optional[List[int]] = None
+    lens: Optional[List[int]] = None
+    slots_of: Optional[Callable[[int, int, int], "np.ndarray"]] = None
     # context parallelism: this rank holds one chunk of every sequence; K/V are gathered over cp_group
     cp_group: Any = None
     extras: Dict[str, Any] = field(default_factory=dict)
+
+    def visible_context(self, window: Optional[int]) -> Tuple[Optional[torch.Tensor], torch.Tensor]:
+        """(flat cache slots of every key the step's tokens can see, packed by sequence; their offsets [B + 1]).  The
+        slots are None when the step's own tokens are all there is.  Layers with the same window share the answer."""
+        if not self.starts or not any(self.starts):
+            return None, self.cu_seqlens
+        key = ("visible", window)
+        if key not in self.extras:
+            parts, cu = [], [0]
+            for b, (start, n) in enumerate(zip(self.starts, self.lens)):
+                lo = max(0, start - window + 1) if window else 0
+                parts.append(self.slots_of(b, lo, start + n))
+                cu.append(cu[-1] + start + n - lo)
+            dev = self.cu_seqlens.device
+            self.extras[key] = (torch.from_numpy(np.concatenate(parts).astype(np.int32)).to(dev),
+                                torch.tensor(cu, dtype=torch.int32).to(dev))
+        return self.extras[key]
 
 
 class YvAttention(nn.Module):

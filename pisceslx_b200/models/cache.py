@@ -4,7 +4,8 @@ The reference keeps Python lists of per-layer block objects and concatenates the
 (model/core/cache.py:535-868, read path :824-835); its unified manager is lossy by default (H2O,
 quantisation, eviction; cache.py:1886-2038).  Here the cache is two device tensors per layer
 ``[num_blocks, block_size, n_kv_head, head_dim]`` plus an int32 block table per sequence; the decode kernel
-reads pages in place.  The cache is exact; eviction policies (LRU of whole sequences, sliding window)
+reads pages in place.  ``YvPagedLatentCache`` keeps the same pages, tables and free list with one latent row per token
+and layer instead of keys and values, and gives pages back once every layer's window has passed them.  The cache is exact; eviction policies (LRU of whole sequences, sliding window)
 are opt-in helpers that only edit block tables.
 """
 from __future__ import annotations
@@ -12,7 +13,11 @@ from __future__ import annotations
 from dataclasses import dataclass
 from typing import Dict, List, Optional, Tuple
 
+import numpy as np
 import torch
+
+
+RELEASED = -1      # table entry of a page that was given back because no later token can see it
 
 
 @dataclass
@@ -66,6 +71,8 @@ class YvPagedKVCache:
         self.tables: Dict[int, List[int]] = {}       # seq id -> physical blocks
         self.lengths: Dict[int, int] = {}
         self.layer_offset = 0                         # first global layer index held by this pipeline stage
+        # tokens (the query's own included) that the widest layer still reads; None = every token stays addressable
+        self.reach: Optional[int] = None
 
     def layer(self, idx: int) -> Tuple[torch.Tensor, torch.Tensor]:
         return self.k[idx - self.layer_offset], self.v[idx - self.layer_offset]
@@ -80,12 +87,30 @@ class YvPagedKVCache:
 
     def free_sequence(self, seq_id: int) -> None:
         for b in self.tables.pop(seq_id, []):
-            self.alloc.release(b)
+            if b != RELEASED:
+                self.alloc.release(b)
         self.lengths.pop(seq_id, None)
+
+    def release_passed(self, seq_id: int) -> int:
+        """Give back the pages that no token from here on can see (all layers windowed; see ``reach``).  Their table
+        entries stay as placeholders, so that page i keeps holding tokens ``i * block_size ...``.  One page of slack
+        is kept for callers that step back a few tokens.  Returns the number of pages freed."""
+        if self.reach is None:
+            return 0
+        bs, tbl = self.cfg.block_size, self.tables[seq_id]
+        last = (self.lengths[seq_id] - self.reach + 1 - bs) // bs          # pages below this one are out of reach
+        freed = 0
+        for i in range(min(last, len(tbl)) - 1, -1, -1):
+            if tbl[i] == RELEASED:
+                break                                                     # everything in front of it has gone before
+            self.alloc.release(tbl[i])
+            tbl[i] = RELEASED
+            freed += 1
+        return freed
 
     def fork(self, src: int, dst: int) -> None:
         """Share all full blocks of ``src`` with ``dst`` (prefix caching / beam search)."""
-        self.tables[dst] = [self.alloc.share(b) for b in self.tables[src]]
+        self.tables[dst] = [b if b == RELEASED else self.alloc.share(b) for b in self.tables[src]]
         self.lengths[dst] = self.lengths[src]
 
     def can_append(self, seq_id: int, n_tokens: int) -> bool:
@@ -101,6 +126,7 @@ class YvPagedKVCache:
     def append_slots(self, seq_id: int, n_tokens: int) -> List[int]:
         """Reserve room for ``n_tokens`` new tokens; returns their flat slot ids (block * block_size + offset)."""
         bs = self.cfg.block_size
+        self.release_passed(seq_id)
         for _ in range(self._blocks_needed(seq_id, n_tokens)):
             self.tables[seq_id].append(self.alloc.alloc())
         start = self.lengths[seq_id]
@@ -108,6 +134,15 @@ class YvPagedKVCache:
         slots = [tbl[(start + i) // bs] * bs + (start + i) % bs for i in range(n_tokens)]
         self.lengths[seq_id] = start + n_tokens
         return slots
+
+    def slots(self, seq_id: int, lo: int, hi: int) -> np.ndarray:
+        """Flat slot ids of the tokens lo .. hi - 1 (which must not have been given back)."""
+        bs = self.cfg.block_size
+        pos = np.arange(lo, hi)
+        pages = np.asarray(self.tables[seq_id], dtype=np.int64)[pos // bs]
+        if pages.size and int(pages.min()) < 0:
+            raise IndexError(f"sequence {seq_id}: tokens {lo}..{hi - 1} reach into released pages")
+        return pages * bs + pos % bs
 
     def block_table_tensor(self, seq_ids: List[int], width: Optional[int] = None) -> torch.Tensor:
         width = width or max(1, max(len(self.tables[s]) for s in seq_ids))
@@ -131,16 +166,43 @@ class YvPagedKVCache:
     def load_state(self, st: Dict[str, object]) -> None:
         self.tables = {int(k): list(v) for k, v in st["tables"].items()}      # type: ignore[union-attr]
         self.lengths = {int(k): int(v) for k, v in st["lengths"].items()}     # type: ignore[union-attr]
-        used = {b for t in self.tables.values() for b in t}
+        used = {b for t in self.tables.values() for b in t if b != RELEASED}
         self.alloc = YvBlockAllocator(self.cfg.num_blocks)
         self.alloc.free = [b for b in range(self.cfg.num_blocks - 1, -1, -1) if b not in used]
         self.alloc.refs = {b: sum(b in t for t in self.tables.values()) for b in used}
-        for i in range(self.n_layer):
-            self.k[i].copy_(st["k"][i])                                        # type: ignore[index]
-            self.v[i].copy_(st["v"][i])                                        # type: ignore[index]
+        for mine, saved in ((self.k, st["k"]), (self.v, st["v"])):
+            for t, src in zip(mine, saved):                                    # type: ignore[arg-type]
+                t.copy_(src)
+
+
+class YvPagedLatentCache(YvPagedKVCache):
+    """Pages of latent rows: layer i stores ``row_sizes[i]`` numbers per token, ``[num_blocks, block_size, row]``."""
+
+    def __init__(self, row_sizes: List[int], cfg: YvCacheConfig, device: torch.device, reach: Optional[int] = None):
+        self.cfg, self.device = cfg, device
+        self.n_layer, self.hk, self.d = len(row_sizes), 1, max(row_sizes)
+        self.k = [torch.zeros(cfg.num_blocks, cfg.block_size, r, dtype=cfg.dtype, device=device) for r in row_sizes]
+        self.v = []
+        self.alloc = YvBlockAllocator(cfg.num_blocks)
+        self.tables, self.lengths = {}, {}
+        self.layer_offset = 0
+        self.reach = reach
+
+    def rows(self, idx: int) -> torch.Tensor:
+        return self.k[idx - self.layer_offset]
+
+    def layer(self, idx: int):
+        raise TypeError("a latent cache has no separate keys and values: use rows()")
+
+    def bytes(self) -> int:
+        return sum(t.numel() * t.element_size() for t in self.k)
 
 
 def cache_for_model(cfg, device: torch.device, num_blocks: int, block_size: Optional[int] = None, tp_size: int = 1,
                     n_layer: Optional[int] = None, dtype: torch.dtype = torch.bfloat16) -> YvPagedKVCache:
     cc = YvCacheConfig(block_size=block_size or cfg.kv_cache_block_size, num_blocks=num_blocks, dtype=dtype)
+    if cfg.layer_specs:
+        from .registry import latent_cache_layout
+        rows, reach = latent_cache_layout(cfg)
+        return YvPagedLatentCache(rows, cc, device, reach)
     return YvPagedKVCache(n_layer or cfg.n_layer, cfg.n_kv_head // tp_size, cfg.head_dim, cc, device)

@@ -15,6 +15,8 @@ from typing import Dict, Iterable, List, Optional, Tuple
 
 import torch
 
+from .cache import RELEASED
+
 
 @dataclass
 class _Entry:
@@ -188,7 +190,7 @@ class YvPrefixCache:
     def publish(self, seq_id: int, tokens: List[int]) -> None:
         """Index the full blocks of a prefilled sequence (the index holds its own reference on each block)."""
         for i, key in enumerate(self._keys(tokens)):
-            if key not in self.index and i < len(self.cache.tables[seq_id]):
+            if key not in self.index and i < len(self.cache.tables[seq_id]) and self.cache.tables[seq_id][i] != RELEASED:
                 self.index[key] = self.cache.alloc.share(self.cache.tables[seq_id][i])
 
     def evict(self, n: int = 1) -> None:

@@ -142,9 +142,12 @@ def _tp_size(model) -> int:
     return par.tp_size if par is not None else 1
 
 
-def _prefill(model, ids: torch.Tensor, cache: YvPagedKVCache, seq_ids: List[int]) -> torch.Tensor:
-    """Run the prompt(s) [B, S] through the model, filling the cache; returns last-token logits [B, V].
+def _prefill(model, ids: torch.Tensor, cache: YvPagedKVCache, seq_ids: List[int],
+             want: Optional[List[int]] = None) -> Optional[torch.Tensor]:
+    """Run the prompt(s), or the next portion of the prompt(s), [B, S] through the model, filling the cache; returns
+    last-token logits [B, V], or with ``want`` the logits at those places of one sequence's portion [len(want), V] (None when the list is empty).
 
+    A portion continues where the sequence's cache ends (models with ``supports_portions``).
     Under tensor parallelism the token rows are sharded over the ranks between the layers (sequence parallel), so the
     row count must divide by the group size: the prompts are padded at the END with tokens that are not cached
     (slot -1); causal attention keeps them out of every real token's context."""
@@ -153,13 +156,26 @@ def _prefill(model, ids: torch.Tensor, cache: YvPagedKVCache, seq_ids: List[int]
     pad = (-S) % _tp_size(model)
     if pad:
         ids = torch.cat([ids, ids.new_zeros(B, pad)], dim=1)
+    starts = [cache.lengths[s] for s in seq_ids]
     ctx = trunk.build_context(B, S + pad, ids.device)
+    if any(starts):
+        if not getattr(model, "supports_portions", False):
+            raise ValueError("this model's attention does not continue a prompt from the cache")
+        ctx.starts, ctx.lens = starts, [S] * B
+        ctx.slots_of = lambda b, lo, hi: cache.slots(seq_ids[b], lo, hi)
+        first = torch.tensor(starts, dtype=torch.int32).to(ids.device)
+        ctx.positions = ctx.positions + first.repeat_interleave(S + pad)
+        ctx.max_position = max(starts) + S + pad
     slots: List[int] = []
     for s in seq_ids:
         slots += cache.append_slots(s, S) + [-1] * pad
     ctx.cache = cache
     ctx.slot_map = torch.tensor(slots, dtype=torch.int32).to(ids.device)
+    if want is not None and B != 1:
+        raise ValueError("wanted places are given for one sequence at a time")
     out = model(input_ids=ids, ctx=ctx, return_logits=False, return_hidden=True)
+    if want is not None:
+        return model.logits(out["hidden_states"][0, want, :]) if want else None
     return model.logits(out["hidden_states"][:, S - 1, :])
 
 
@@ -186,7 +202,8 @@ def _decode_step(model, tokens: torch.Tensor, cache: YvPagedKVCache, seq_ids: Li
     ctx = AttnContext(positions=pos, cu_seqlens=torch.arange(Bp + 1, dtype=torch.int32, device=dev), max_len=1,
                       cos=cos, sin=sin, causal=True, cache=cache,
                       slot_map=torch.tensor(slots, dtype=torch.int32).to(dev),
-                      block_table=table, seq_lens=lens, decode=True)
+                      block_table=table, seq_lens=lens, decode=True,
+                      max_position=max(cache.lengths[s] for s in seq_ids))
     out = model(input_ids=tokens.view(Bp, 1), ctx=ctx, return_logits=False, return_hidden=True)
     return model.logits(out["hidden_states"][:B, -1, :])
 

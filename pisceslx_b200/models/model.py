@@ -24,6 +24,7 @@ from ..ops.loss import linear_cross_entropy
 from .attention import AttnContext
 from .blocks import YvTransformerBlock
 from .norms import YvRMSNorm, YvRotaryEmbedding
+from .registry import model_class
 
 
 class YvModelOutput(dict):
@@ -39,7 +40,32 @@ class YvModelOutput(dict):
         self[k] = v
 
 
-class YvModel(nn.Module):
+class YvPackedTrunk(nn.Module):
+    """What every trunk shares: packed sequences described by an ``AttnContext``.  Subclasses set ``rotary``: one table
+    for all layers, or None when the layers bring their own."""
+
+    def build_context(self, batch: int, seq: int, device: torch.device, lengths: Optional[torch.Tensor] = None,
+                      causal: bool = True) -> AttnContext:
+        """Context for ``batch`` sequences of equal length ``seq`` (or the given per-sequence lengths)."""
+        if lengths is None:
+            cu = torch.arange(0, (batch + 1) * seq, seq, dtype=torch.int32, device=device)
+            pos = torch.arange(seq, dtype=torch.int32, device=device).repeat(batch)
+            max_len = seq
+        else:
+            cu = torch.zeros(batch + 1, dtype=torch.int32, device=device)
+            cu[1:] = torch.cumsum(lengths.int(), 0)
+            total = int(cu[-1].item())
+            seq_id = torch.repeat_interleave(torch.arange(batch, device=device), lengths.long())
+            pos = (torch.arange(total, device=device) - cu[:-1].long()[seq_id]).int()
+            max_len = int(lengths.max().item())
+        cos = sin = None
+        if self.rotary is not None:
+            cos, sin = self.rotary.tables(max_len, device)
+        return AttnContext(positions=pos, cu_seqlens=cu, max_len=max_len, cos=cos, sin=sin, causal=causal,
+                           max_position=max_len)
+
+
+class YvModel(YvPackedTrunk):
     def __init__(self, cfg: YvConfig, parallel=None):
         super().__init__()
         self.cfg, self.parallel = cfg, parallel
@@ -94,25 +120,6 @@ class YvModel(nn.Module):
         setattr(self, name, module)
         if name not in self.materialized_components:
             self.materialized_components.append(name)
-
-    def build_context(self, batch: int, seq: int, device: torch.device, lengths: Optional[torch.Tensor] = None,
-                      causal: bool = True) -> AttnContext:
-        """Context for ``batch`` sequences of equal length ``seq`` (or the given per-sequence lengths)."""
-        if lengths is None:
-            cu = torch.arange(0, (batch + 1) * seq, seq, dtype=torch.int32, device=device)
-            pos = torch.arange(seq, dtype=torch.int32, device=device).repeat(batch)
-            max_len = seq
-        else:
-            cu = torch.zeros(batch + 1, dtype=torch.int32, device=device)
-            cu[1:] = torch.cumsum(lengths.int(), 0)
-            total = int(cu[-1].item())
-            seq_id = torch.repeat_interleave(torch.arange(batch, device=device), lengths.long())
-            pos = (torch.arange(total, device=device) - cu[:-1].long()[seq_id]).int()
-            max_len = int(lengths.max().item())
-        cos = sin = None
-        if self.rotary is not None:
-            cos, sin = self.rotary.tables(max_len, device)
-        return AttnContext(positions=pos, cu_seqlens=cu, max_len=max_len, cos=cos, sin=sin, causal=causal)
 
     def embed_tokens(self, input_ids: torch.Tensor, attention_mask: Optional[torch.Tensor] = None) -> torch.Tensor:
         h = self.embed(input_ids)
@@ -185,10 +192,13 @@ class YvModel(nn.Module):
 
 
 class YvModelForCausalLM(nn.Module):
+    trunk_class: type = YvModel
+    supports_portions = False         # attention of a prompt's later portion over cached earlier ones
+
     def __init__(self, cfg: YvConfig, parallel=None):
         super().__init__()
         self.cfg, self.parallel = cfg, parallel
-        self.model = YvModel(cfg, parallel)
+        self.model = self.trunk_class(cfg, parallel)
         self.tied = cfg.tie_word_embeddings and self.model.is_first_stage and self.model.is_last_stage
         if self.model.is_last_stage and not self.tied:
             self.lm_head = nn.Parameter(torch.empty(cfg.vocab_size, cfg.hidden_size))
@@ -441,7 +451,7 @@ def build_model(cfg: YvConfig, device: Optional[torch.device | str] = None, dtyp
     try:
         torch.set_default_dtype(dtype)
         with torch.device(device):
-            model = YvModelForCausalLM(cfg, parallel)
+            model = model_class(cfg)(cfg, parallel)
     finally:
         torch.set_default_dtype(prev)
     # routing state stays fp32 regardless of the parameter dtype

@@ -67,21 +67,26 @@ class YvRotaryEmbedding(nn.Module):
     """cos/sin tables for rotate-half RoPE with optional linear / dynamic-NTK / YaRN scaling."""
 
     def __init__(self, rot_dim: int, max_position: int = 8192, theta: float = 1e4, scaling_type: str = "none",
-                 scaling_factor: float = 1.0, original_max_position: Optional[int] = None):
+                 scaling_factor: float = 1.0, original_max_position: Optional[int] = None,
+                 yarn: Optional[Dict[str, float]] = None):
+        """``yarn`` overrides the YaRN constants: ``beta_fast`` / ``beta_slow`` (turns over the original range that
+        bound the ramp), ``ramp_end`` (the largest end of the ramp) and ``magnitude`` (factor on cos and sin)."""
         super().__init__()
         self.rot_dim, self.theta = rot_dim, theta
+        self.yarn = dict(yarn or {})
         self.scaling_type, self.scaling_factor = scaling_type, scaling_factor
         self.original_max = original_max_position or max_position
         self.max_position = 0
         self.register_buffer("cos", torch.empty(0), persistent=False)
         self.register_buffer("sin", torch.empty(0), persistent=False)
+        self._retired: list = []
         self._build(max_position, torch.device("cpu"))
 
     def _build(self, max_position: int, device: torch.device) -> None:
         theta = self.theta
-        if self.scaling_type == "yarn" and self.scaling_factor > 1:
+        if self.scaling_type == "yarn" and (self.scaling_factor > 1 or self.yarn):
             cos, sin = ref.yarn_tables(max_position, self.rot_dim, theta, self.scaling_factor, self.original_max,
-                                       device=device)
+                                       device=device, **self.yarn)
         else:
             lin = 1.0
             if self.scaling_type == "linear":
@@ -91,6 +96,8 @@ class YvRotaryEmbedding(nn.Module):
                 theta = theta * (self.scaling_factor * s - (self.scaling_factor - 1)) ** (
                     self.rot_dim / max(self.rot_dim - 2, 1))
             cos, sin = ref.rope_tables(max_position, self.rot_dim, theta, lin, device=device)
+        if self.cos.is_cuda:
+            self._retired.append((self.cos, self.sin))       # captured decode steps keep reading the table they saw
         self.cos, self.sin = cos, sin
         self.max_position = max_position
 

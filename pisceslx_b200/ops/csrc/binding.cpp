@@ -131,8 +131,11 @@ void gemm_grouped_k(const Tensor& a, const Tensor& b, Tensor c, const Tensor& se
 void gemm_batched(const Tensor& a, const Tensor& b, Tensor c, bool a_mn, bool b_mn, bool accumulate, int64_t bn,
                   const c10::optional<Tensor>& status, bool symmetric) {
   check_bf16(a, "a"); check_bf16(b, "b"); check_cuda(c, "c");
-  TORCH_CHECK(a.dim() == 3 && b.dim() == 3 && c.dim() == 3 && a.is_contiguous() && b.is_contiguous() &&
-              c.is_contiguous(), "gemm_batched: contiguous 3-D operands expected");
+  // groups are stacked along the rows: a row pitch is allowed, a gap between groups is not
+  auto stacked = [](const Tensor& t) {
+    return t.dim() == 3 && t.stride(2) == 1 && (t.size(0) == 1 || t.stride(0) == t.size(1) * t.stride(1));
+  };
+  TORCH_CHECK(stacked(a) && stacked(b) && stacked(c), "gemm_batched: stacked 3-D operands expected");
   TORCH_CHECK(a.size(0) == b.size(0) && a.size(0) == c.size(0), "gemm_batched: batch sizes differ");
   const c10::cuda::CUDAGuard guard(a.device());
   yv::GemmArgs g;
@@ -145,6 +148,7 @@ void gemm_batched(const Tensor& a, const Tensor& b, Tensor c, bool a_mn, bool b_
   g.N = static_cast<int>(b_mn ? b.size(2) : b.size(1));
   TORCH_CHECK((b_mn ? b.size(1) : b.size(2)) == g.K, "gemm_batched: K mismatch");
   TORCH_CHECK(c.size(1) == g.M && c.size(2) == g.N, "gemm_batched: output shape mismatch");
+  g.lda = a.stride(1); g.ldb = b.stride(1); g.ldc = c.stride(1);
   g.out_fp32 = dt_code(c);
   g.accumulate = accumulate ? 1 : 0;
   g.bn = static_cast<int>(bn);

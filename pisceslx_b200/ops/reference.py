@@ -50,8 +50,12 @@ def rope_tables(max_pos: int, rot_dim: int, theta: float = 1e4, scaling: float =
 
 def yarn_tables(max_pos: int, rot_dim: int, theta: float, factor: float, original_max: int,
                 beta_fast: float = 32.0, beta_slow: float = 1.0,
-                device: Optional[torch.device] = None) -> Tuple[torch.Tensor, torch.Tensor]:
-    """YaRN: interpolate low frequencies by ``factor``, keep high ones, blend in between."""
+                device: Optional[torch.device] = None,
+                ramp_end: Optional[int] = None,
+                magnitude: Optional[float] = None) -> Tuple[torch.Tensor, torch.Tensor]:
+    """YaRN: interpolate low frequencies by ``factor``, keep high ones, blend in between.  ``ramp_end`` bounds the
+    upper end of the ramp (default: the last pair); ``magnitude`` multiplies cos and sin (default: 0.1 ln factor + 1
+    above a factor of 1)."""
     half = rot_dim // 2
     idx = torch.arange(0, half, dtype=torch.float64)
     inv = 1.0 / (theta ** (idx * 2.0 / rot_dim))
@@ -59,11 +63,11 @@ def yarn_tables(max_pos: int, rot_dim: int, theta: float, factor: float, origina
     def corr(n_rot: float) -> float:
         return rot_dim * math.log(original_max / (n_rot * 2 * math.pi)) / (2 * math.log(theta))
 
-    lo, hi = max(math.floor(corr(beta_fast)), 0), min(math.ceil(corr(beta_slow)), half - 1)
+    lo, hi = max(math.floor(corr(beta_fast)), 0), min(math.ceil(corr(beta_slow)), half - 1 if ramp_end is None else ramp_end)
     ramp = ((idx - lo) / max(hi - lo, 1e-3)).clamp(0, 1)
     inv = inv / factor * ramp + inv * (1 - ramp)
     ang = torch.outer(torch.arange(max_pos, dtype=torch.float64), inv)
-    m = 0.1 * math.log(factor) + 1.0 if factor > 1 else 1.0
+    m = magnitude if magnitude is not None else 0.1 * math.log(factor) + 1.0 if factor > 1 else 1.0
     return (ang.cos() * m).float().to(device), (ang.sin() * m).float().to(device)
 
 
@@ -77,6 +81,46 @@ def apply_rope(x: torch.Tensor, cos: torch.Tensor, sin: torch.Tensor, positions:
     a, b, rest = xf[..., :half], xf[..., half:rot_dim], xf[..., rot_dim:]
     out = torch.cat([a * c - b * s, b * c + a * s, rest], dim=-1)
     return out.to(x.dtype)
+
+
+def latent_attention(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, kr: torch.Tensor, gate: Optional[torch.Tensor],
+                     cu_q: torch.Tensor, cu_k: torch.Tensor, heads: int, window: Optional[int],
+                     scale: float) -> torch.Tensor:
+    """Windowed causal attention with a key part ``kr`` shared by the heads and a per-head sigmoid output gate."""
+    outs = []
+    cq, ck = cu_q.tolist(), cu_k.tolist()
+    for b in range(len(cq) - 1):
+        nq, nk = cq[b + 1] - cq[b], ck[b + 1] - ck[b]
+        qs = q[cq[b]:cq[b + 1]].float().view(nq, heads, -1)
+        ks = k[ck[b]:ck[b + 1]].float().view(nk, heads, -1)
+        vs = v[ck[b]:ck[b + 1]].float().view(nk, heads, -1)
+        ks = torch.cat([ks, kr[ck[b]:ck[b + 1]].float().unsqueeze(1).expand(-1, heads, -1)], -1)
+        i = torch.arange(nq, device=q.device)[:, None] + (nk - nq)
+        d = i - torch.arange(nk, device=q.device)[None, :]
+        ok = (d >= 0) & (d < window) if window else d >= 0
+        sc = torch.einsum("qhd,khd->hqk", qs, ks) * scale
+        w = torch.softmax(sc.masked_fill(~ok, float("-inf")), -1)
+        o = torch.einsum("hqk,khd->qhd", w, vs)
+        if gate is not None:
+            o = o * torch.sigmoid(gate[cq[b]:cq[b + 1]].float()).unsqueeze(-1)
+        outs.append(o.reshape(nq, -1))
+    return torch.cat(outs, 0).to(q.dtype)
+
+
+def latent_decode(q_lat: torch.Tensor, cache: torch.Tensor, kv_rank: int, block_table: torch.Tensor,
+                  seq_lens: torch.Tensor, window: Optional[int], scale: float) -> torch.Tensor:
+    """q_lat [heads, R, row] against the paged latent rows -> weighted latents [heads, R, kv_rank]."""
+    heads, R, row = q_lat.shape
+    block = cache.shape[1]
+    out = torch.zeros(heads, R, kv_rank, dtype=q_lat.dtype, device=q_lat.device)
+    for b, n in enumerate(seq_lens.tolist()):
+        first = max(0, n - window) if window else 0
+        pos = torch.arange(first, n)
+        slots = block_table[b].long()[pos // block] * block + pos % block
+        c = cache.view(-1, row)[slots].float()
+        w = torch.softmax((q_lat[:, b].float() @ c.t()) * scale, -1)
+        out[:, b] = (w @ c[:, :kv_rank]).to(out.dtype)
+    return out
 
 
 def apply_rope3d(x: torch.Tensor, pos_thw: torch.Tensor, sections: Sequence[int], theta: float = 1e4) -> torch.Tensor:

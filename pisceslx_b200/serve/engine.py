@@ -54,6 +54,8 @@ class YvEngineConfig:
     use_cuda_graphs: bool = True          # replay decode steps from CUDA graphs (one graph per batch bucket)
     graph_max_seq_len: int = 8192         # sequences longer than this decode through the eager step
     status_check_steps: int = 16          # read the kernels' status word every this many decode steps (0 = never)
+    prefill_portion: int = 0              # run prompts in portions of at most this many tokens (0 = whole; models
+                                          # that continue a prompt from the cache only)
 
 
 class YvInferenceEngine:
@@ -154,12 +156,35 @@ class YvInferenceEngine:
         self.cache.add_sequence(req.request_id)
         self._reserved[req.request_id] = self._worst_case_blocks(req)
         context = req.prompt_ids + req.output_ids           # non-empty output: resuming after a preemption
-        ids = torch.tensor([context], dtype=torch.long, device=self.device)
-        logits = _prefill(self.model, ids, self.cache, [req.request_id])
+        logits = self.run_tokens(req.request_id, context, [len(context) - 1])
         self.stats["prefill_tokens"] += len(context)
+        ids = torch.tensor([context], dtype=torch.long, device=self.device)
         tok = int(YvSampler(req.sampling).sample(logits, ids)[0])
         self.running.append(req)
         self._emit(req, tok)
+
+    # ---- the model step behind prompts, resumed requests and replayed traces ----------------------------------
+    @torch.no_grad()
+    def run_tokens(self, seq_id: int, tokens: List[int], want: List[int]) -> Optional[torch.Tensor]:
+        """Append ``tokens`` to a cached sequence (``cache.add_sequence`` first) and return the fp32 logits at the
+        places ``want`` among them [len(want), V] (None when nothing is wanted).  A single token of a started sequence
+        is a decode step; anything else runs as prompt portions of at most ``prefill_portion`` tokens."""
+        if len(tokens) == 1 and self.cache.lengths[seq_id] > 0:
+            logits = self.graph.step(list(tokens), [seq_id])
+            return logits[[0] * len(want)] if want else None
+        size = self.cfg.prefill_portion if getattr(self.model, "supports_portions", False) else 0
+        size = size or len(tokens)
+        order = sorted(set(want))
+        parts = []
+        for lo in range(0, len(tokens), size):
+            part = tokens[lo:lo + size]
+            here = [w - lo for w in order if lo <= w < lo + len(part)]
+            ids = torch.tensor([part], dtype=torch.long, device=self.device)
+            parts.append(_prefill(self.model, ids, self.cache, [seq_id], want=here))
+        if not want:
+            return None
+        logits = torch.cat([p for p in parts if p is not None], 0)
+        return logits if order == list(want) else logits[[order.index(w) for w in want]]
 
     # ---- one scheduler iteration ---------------------------------------------------------------------------
     @torch.no_grad()

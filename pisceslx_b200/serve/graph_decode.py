@@ -88,7 +88,7 @@ class YvDecodeGraphRunner:
         B = bk.B
         ctx = AttnContext(positions=bk.meta[1], cu_seqlens=self._cu[: B + 1], max_len=1, cos=self._cos, sin=self._sin,
                           causal=True, cache=self.cache, slot_map=bk.meta[2], block_table=bk.table,
-                          seq_lens=bk.meta[3], decode=True)
+                          seq_lens=bk.meta[3], decode=True, max_position=self.max_seq_len)
         out = self.model(input_ids=bk.meta[0].long().view(B, 1), ctx=ctx, return_logits=False, return_hidden=True)
         return self.model.logits(out["hidden_states"][:, -1, :])
 
