@@ -215,7 +215,8 @@ class PiscesLxInferOrchestrator:
         if args.dry_run:
             print(json.dumps({"prompt_tokens": len(YvTokenizer.instance().encode(args.prompt)), "model_size": args.model_size}))
             return 0
-        model = load_model_for_inference(args.model_size, args.ckpt, args.device, args.model_config)
+        dtype = {"bf16": torch.bfloat16, "fp32": torch.float32}.get(getattr(args, "dtype", None))
+        model = load_model_for_inference(args.model_size, args.ckpt, args.device, args.model_config, dtype)
         tok = YvTokenizer.for_vocab(model.cfg.vocab_size)
         ids = torch.tensor([tok.encode(args.prompt)], dtype=torch.long, device=next(model.parameters()).device)
         ids = ids.clamp_(0, model.cfg.vocab_size - 1)

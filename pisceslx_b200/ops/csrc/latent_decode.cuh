@@ -1,7 +1,461 @@
+// Decode in the latent space on the tensor cores: every head of a sequence attends over the same cached rows
+// [latent | rotated key part], which are keys with all their columns and values with the latent ones.
+//
+// A tile is one cache page of 64 tokens, stored in shared memory as slabs of 64 columns (128-byte swizzle) and used
+// twice from there:
+//   S[128 heads, 64 keys]   = Q[heads, row] * C[64 keys, row]^T            (SS, both K-major; NH rows of Q are real)
+//   O^T[128 dims, NH heads] += C^T[dims, 64 keys] * P[NH heads, 64 keys]^T  (SS, A MN-major), one product per 128 dims
+// The M dimension of the first product reads past the NH real rows of Q into whatever follows in shared memory; those
+// lanes of S are never read.
+//
+// grid = (head groups of NH, sequences, key ranges), 160 threads:
+//   warps 0..3  softmax: thread t owns head t (TMEM lane t of S, no cross-lane reductions); O^T is rescaled by all
+//               128 threads (lane = latent dimension) when a head's reference maximum moves, which is rare
+//   warp 4      one lane issues the TMA copies and both products
+// The page slabs travel through a ring counted in slabs, so that a part of the page after next is already in flight
+// when two whole pages do not leave room for a third.  A page takes an even number of ring slots: the pair of slabs
+// behind one 128-row product is always contiguous.
+// Output: normalised bf16 when there is one key range, otherwise (max, sum, fp32 sums) per range, merged below.
 #pragma once
 #include "latent_ops.h"
+#include "per_device.h"
 #include "sm100.cuh"
+#include "tensormap.h"
+
 namespace yv {
-inline int launch_latent_decode_mma(const LatentDecodeArgs&, cudaStream_t) { return -99; }
-bool latent_decode_on_tensor_cores(const LatentDecodeArgs&) { return false; }
+
+struct LatentDecodeParams {
+  CUtensorMap tma_c;               // 2-D (row, token slot), box (64, 64), 128B swizzle
+  const __nv_bfloat16* q;          // [heads, rows_pad, row]
+  __nv_bfloat16* out;              // [heads, rows_pad, kv_rank]
+  const int* block_table;
+  const int* seq_lens;
+  float* partial_o;
+  float* partial_ml;
+  int64_t rows_pad;
+  int heads, kv_rank, row, max_blocks, num_blocks, window, splits;
+  int slabs, slots, ring, chunks;  // slabs and ring slots per page, ring size in slabs, 128-dim chunks of the latent
+  uint32_t tmem_cols;
+  float scale_log2;
+  uint32_t* status;
+};
+
+constexpr int kLdThreads = 160;
+constexpr int kLdKeys = 64;
+constexpr int kLdSlab = kLdKeys * 128;
+constexpr int kLdBars = 4;                                  // pages whose arrival can be tracked at a time
+constexpr int kLdSmemMax = 227 * 1024;
+constexpr int kLdTableCap = 512;                            // block-table entries of a key range staged in shared memory
+constexpr int kLdStatic = 4096;                             // bound on the kernel's static shared memory
+
+// Barrier over the 128 softmax threads with an OR of `v`.  The instruction is warp-aligned: lanes that left a bounded
+// wait at different times are brought together first.
+__device__ __forceinline__ bool ld_barrier_or(bool v) {
+  uint32_t r;
+  __syncwarp();
+  asm volatile(
+      "{\n"
+      ".reg .pred pin, pout;\n"
+      "setp.ne.u32 pin, %1, 0;\n"
+      "bar.red.or.pred pout, 1, 128, pin;\n"
+      "selp.u32 %0, 1, 0, pout;\n"
+      "}\n"
+      : "=r"(r)
+      : "r"(static_cast<uint32_t>(v))
+      : "memory");
+  return r != 0u;
 }
+
+__device__ __forceinline__ float ld_exp2(float x) {
+  float y;
+  asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+  return y;
+}
+
+template <int NH>
+__global__ void __launch_bounds__(kLdThreads) latent_decode_kernel(const __grid_constant__ LatentDecodeParams p) {
+  constexpr uint32_t kIdescQK = make_idesc_bf16(128, kLdKeys, false, false);
+  constexpr uint32_t kIdescPV = make_idesc_bf16(128, NH, true, false);
+  constexpr int kQSlab = NH * 128;                          // bytes of one 64-column slab of Q (and of one P buffer)
+  extern __shared__ uint8_t ld_raw[];
+  uint8_t* sm = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(ld_raw) + 1023) & ~uintptr_t(1023));
+  uint8_t* sQ = sm;                                         // [slabs][NH][128 B]
+  uint8_t* sP = sQ + p.slabs * kQSlab;                      // [2][NH][128 B]
+  uint8_t* ring = sP + 2 * kQSlab;                          // [ring][64 keys][128 B]
+  __shared__ uint64_t full_bar[kLdBars], s_bar[2], pv_bar[2], p_bar[2];
+  __shared__ uint32_t tmem_slot;
+  __shared__ float s_alpha[2][NH], s_l[NH];
+  __shared__ int s_table[kLdTableCap];
+
+  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+  const int h0 = blockIdx.x * NH, b = blockIdx.y, split = blockIdx.z;
+  int n = p.seq_lens[b];
+  {
+    const int64_t cap = static_cast<int64_t>(p.max_blocks) * kLdKeys;
+    if (n < 0 || n > cap) {
+      if (tid == 0 && p.status != nullptr) atomicOr(p.status, kStatusIndexOutOfRange);
+      n = n < 0 ? 0 : static_cast<int>(cap);
+    }
+  }
+  const int first = (p.window > 0 && n > p.window) ? n - p.window : 0;
+  const int page_lo = first / kLdKeys, page_hi = (n + kLdKeys - 1) / kLdKeys;
+  const int per = (page_hi - page_lo + p.splits - 1) / p.splits;
+  const int pg0 = page_lo + split * per;
+  const int pg1 = min(page_hi, pg0 + per);
+  const int n_tiles = pg1 > pg0 ? pg1 - pg0 : 0;
+  const int* gtable = p.block_table + static_cast<int64_t>(b) * p.max_blocks + pg0;
+  const int* table = n_tiles <= kLdTableCap ? s_table : gtable;       // pages of this key range
+  if (n_tiles <= kLdTableCap)
+    for (int i = tid; i < n_tiles; i += kLdThreads) s_table[i] = gtable[i];
+
+  if (tid == 0) {
+    tma_prefetch_desc(&p.tma_c);
+    for (int i = 0; i < kLdBars; ++i) mbar_init(&full_bar[i], 1);
+    for (int i = 0; i < 2; ++i) { mbar_init(&s_bar[i], 1); mbar_init(&pv_bar[i], 1); mbar_init(&p_bar[i], 128); }
+    fence_barrier_init();
+  }
+  if (warp == 0) {
+    tmem_alloc(&tmem_slot, p.tmem_cols);
+    tmem_relinquish();
+  }
+  // Q as K-major swizzled slabs; heads and columns that do not exist are zero.  P rows are written every tile.
+  for (int i = tid; i < p.slabs * NH * 8; i += kLdThreads) {
+    const int v = i & 7, r = (i >> 3) % NH, c = (i >> 3) / NH;
+    const int col = c * 64 + v * 8;
+    uint4 val = make_uint4(0, 0, 0, 0);
+    if (h0 + r < p.heads && col < p.row)
+      val = *reinterpret_cast<const uint4*>(p.q + (static_cast<int64_t>(h0 + r) * p.rows_pad + b) * p.row + col);
+    *reinterpret_cast<uint4*>(sQ + c * kQSlab + r * 128 + ((v ^ (r & 7)) << 4)) = val;
+  }
+  fence_proxy_async_smem();
+  tc_fence_before_sync();
+  __syncthreads();
+  tc_fence_after_sync();
+  const uint32_t tmem_base = tmem_slot;
+  const uint32_t tO = tmem_base + 128u;                     // S buffers at columns 0 and 64
+
+  if (warp == 4) {
+    // ------------------------------------ issuer ---------------------------------------------
+    if (lane == 0 && n_tiles > 0) {
+      int next = 0;                                         // next ring slot (counted from the first page on) to fill
+      auto fill = [&](int pages_done) {
+        const int limit = min(pages_done * p.slots + p.ring, n_tiles * p.slots);
+        for (; next < limit; ++next) {
+          const int j = next / p.slots, c = next - j * p.slots;
+          // a page of arrivals is tracked by barrier j % kLdBars: its previous user must have been consumed
+          if (j >= pages_done + kLdBars) break;
+          if (c == 0) mbar_expect_tx(&full_bar[j % kLdBars], static_cast<uint32_t>(p.slabs) * kLdSlab);
+          if (c >= p.slabs) continue;
+          int page = table[j];
+          if (page < 0 || page >= p.num_blocks) {           // reported; its keys are masked by the softmax warps
+            if (p.status != nullptr) atomicOr(p.status, kStatusIndexOutOfRange);
+            page = 0;
+          }
+          tma_load_2d(ring + static_cast<size_t>(next % p.ring) * kLdSlab, &p.tma_c, &full_bar[j % kLdBars], c * 64,
+                      page * kLdKeys);
+        }
+      };
+      const int steps = (p.row + 15) / 16;
+      const uint32_t aQ = smem_u32(sQ), aR = smem_u32(ring), aP = smem_u32(sP);
+      auto slab_addr = [&](int j, int c) { return aR + static_cast<uint32_t>((j * p.slots + c) % p.ring) * kLdSlab; };
+      auto issue_qk = [&](int j) -> bool {
+        if (!mbar_wait(&full_bar[j % kLdBars], (j / kLdBars) & 1u, p.status)) return false;
+        tc_fence_after_sync();
+        const uint32_t dS = tmem_base + static_cast<uint32_t>((j & 1) * 64);
+        for (int kk = 0; kk < steps; ++kk) {
+          const int c = kk >> 2, o = (kk & 3) * 32;
+          tc_mma_f16_ss(dS, make_smem_desc(aQ + c * kQSlab + o, 16, 1024), make_smem_desc(slab_addr(j, c) + o, 16, 1024),
+                        kIdescQK, kk != 0 ? 1u : 0u);
+        }
+        tc_commit(&s_bar[j & 1]);
+        return true;
+      };
+      fill(0);
+      bool ok = issue_qk(0);
+      for (int j = 0; j < n_tiles && ok; ++j) {
+        bool ahead = j + 1 >= n_tiles;
+        if (!ahead && next >= (j + 1) * p.slots + p.slabs) {      // the next page is on its way: score it now
+          ok = issue_qk(j + 1);
+          ahead = true;
+          if (!ok) break;
+        }
+        if (j > 0) {
+          ok = mbar_wait(&pv_bar[(j - 1) & 1], ((j - 1) >> 1) & 1u, p.status);
+          if (!ok) break;
+          fill(j);                                                // pages 0 .. j - 1 have been consumed
+        }
+        if (!ahead) {
+          ok = issue_qk(j + 1);
+          if (!ok) break;
+        }
+        // (one barrier per P buffer: the softmax warps may finish page j + 1 before this thread looks at page j)
+        ok = mbar_wait(&p_bar[j & 1], (j >> 1) & 1u, p.status);
+        if (!ok) break;
+        tc_fence_after_sync();
+        const uint32_t bP = aP + static_cast<uint32_t>((j & 1) * kQSlab);
+        for (int m = 0; m < p.chunks; ++m) {
+          const uint32_t aC = slab_addr(j, 2 * m);
+#pragma unroll
+          for (int kk = 0; kk < kLdKeys / 16; ++kk)
+            tc_mma_f16_ss(tO + static_cast<uint32_t>(m * NH), make_smem_desc(aC + kk * 2048, kLdSlab, 1024),
+                          make_smem_desc(bP + kk * 32, 16, 1024), kIdescPV, (j | kk) != 0 ? 1u : 0u);
+        }
+        tc_commit(&pv_bar[j & 1]);
+      }
+    }
+  } else {
+    // ------------------------------------ softmax --------------------------------------------
+    const uint32_t lane_off = static_cast<uint32_t>(warp * 32) << 16;
+    const bool scoring = warp * 32 < NH;                    // warp-uniform: this warp's lanes hold heads
+    float m_used = -1.0e29f, l_sum = 0.f;
+    bool ok = true;
+    for (int j = 0; j < n_tiles; ++j) {
+      const int page = table[j];
+      const bool page_ok = page >= 0 && page < p.num_blocks;
+      const int k0 = (pg0 + j) * kLdKeys;
+      // P buffer j & 1 was read by the product of page j - 2
+      if (j >= 2) {
+        ok = ok && mbar_wait(&pv_bar[j & 1], ((j - 2) >> 1) & 1u, p.status);
+        ok = __all_sync(0xFFFFFFFFu, ok);
+      }
+      float alpha = 1.f;
+      bool rescale = false;
+      if (scoring) {
+        ok = ok && mbar_wait(&s_bar[j & 1], (j >> 1) & 1u, p.status);
+        ok = __all_sync(0xFFFFFFFFu, ok);
+        if (ok) {
+          tc_fence_after_sync();
+          uint32_t s[64];
+          {
+            uint32_t(&c0)[32] = *reinterpret_cast<uint32_t(*)[32]>(&s[0]);
+            uint32_t(&c1)[32] = *reinterpret_cast<uint32_t(*)[32]>(&s[32]);
+            const uint32_t tS = tmem_base + lane_off + static_cast<uint32_t>((j & 1) * 64);
+            tmem_ld32(tS, c0);
+            tmem_ld32(tS + 32, c1);
+            tc_wait_ld();
+          }
+          float mx = -1.0e30f;
+          if (k0 < first || k0 + kLdKeys > n || !page_ok) {
+#pragma unroll
+            for (int i = 0; i < 64; ++i)
+              if (k0 + i < first || k0 + i >= n || !page_ok) s[i] = 0xFF800000u;
+          }
+#pragma unroll
+          for (int i = 0; i < 64; ++i) mx = fmaxf(mx, __uint_as_float(s[i]));
+          mx = mx > -0.5e30f ? mx * p.scale_log2 : -1.0e30f;
+          if (mx > m_used + 8.f) {                          // lazy: the reference maximum moves in large steps only
+            alpha = ld_exp2(m_used - mx);
+            m_used = mx;
+            rescale = j > 0;
+          }
+          uint32_t pk[32];
+          float ls = 0.f;
+#pragma unroll
+          for (int i = 0; i < 32; ++i) {
+            const float e0 = ld_exp2(fmaf(__uint_as_float(s[2 * i]), p.scale_log2, -m_used));
+            const float e1 = ld_exp2(fmaf(__uint_as_float(s[2 * i + 1]), p.scale_log2, -m_used));
+            const uint32_t bits = pack_bf16(e0, e1);
+            pk[i] = bits;
+            ls += __uint_as_float(bits << 16) + __uint_as_float(bits & 0xFFFF0000u);   // the weights as multiplied
+          }
+          l_sum = l_sum * alpha + ls;
+          const int r = tid;                                // head row
+          if (r < NH) {
+            s_alpha[j & 1][r] = alpha;
+            uint8_t* row = sP + (j & 1) * kQSlab + r * 128;
+#pragma unroll
+            for (int c = 0; c < 8; ++c)
+              *reinterpret_cast<uint4*>(row + ((c ^ (r & 7)) << 4)) =
+                  make_uint4(pk[4 * c], pk[4 * c + 1], pk[4 * c + 2], pk[4 * c + 3]);
+          } else {
+            rescale = false;                                // lanes past NH hold no head
+          }
+          __syncwarp();
+          tc_fence_before_sync();
+        }
+      }
+      if (ld_barrier_or(rescale || !ok)) {
+        ok = !ld_barrier_or(!ok);                           // all 128 threads agree
+        if (!ok) break;
+        // O^T holds sums relative to the old maxima: the previous product must be complete before it is scaled
+        ok = mbar_wait(&pv_bar[(j - 1) & 1], ((j - 1) >> 1) & 1u, p.status);
+        ok = __all_sync(0xFFFFFFFFu, ok);
+        ok = !ld_barrier_or(!ok);
+        if (!ok) break;
+        tc_fence_after_sync();
+        for (int m = 0; m < p.chunks; ++m) {
+#pragma unroll
+          for (int g = 0; g < NH; g += 16) {
+            uint32_t o[16];
+            tmem_ld16(tO + lane_off + static_cast<uint32_t>(m * NH + g), o);
+            tc_wait_ld();
+#pragma unroll
+            for (int i = 0; i < 16; ++i) o[i] = __float_as_uint(__uint_as_float(o[i]) * s_alpha[j & 1][g + i]);
+            tmem_st16(tO + lane_off + static_cast<uint32_t>(m * NH + g), o);
+          }
+        }
+        tc_wait_st();
+        tc_fence_before_sync();
+      }
+      fence_proxy_async_smem();
+      mbar_arrive(&p_bar[j & 1]);
+    }
+    if (ok && n_tiles > 0) ok = mbar_wait(&pv_bar[(n_tiles - 1) & 1], ((n_tiles - 1) >> 1) & 1u, p.status);
+    ok = __all_sync(0xFFFFFFFFu, ok);
+    if (tid < NH) s_l[tid] = l_sum;
+    ok = !ld_barrier_or(!ok);
+    // after a wait that ran out (status set) the outputs are still written, as zeros
+    if (tid < NH && h0 + tid < p.heads && p.splits > 1) {
+      const int64_t base = (static_cast<int64_t>(b) * p.heads + h0 + tid) * p.splits + split;
+      p.partial_ml[base * 2] = ok ? m_used : -1.0e29f;
+      p.partial_ml[base * 2 + 1] = ok ? l_sum : 0.f;
+    }
+    tc_fence_after_sync();
+    for (int m = 0; m < p.chunks; ++m) {
+      const int dim = m * 128 + tid;
+#pragma unroll
+      for (int g = 0; g < NH; g += 16) {
+        uint32_t o[16];
+        __syncwarp();
+        if (ok && n_tiles > 0) {
+          tmem_ld16(tO + lane_off + static_cast<uint32_t>(m * NH + g), o);
+          tc_wait_ld();
+        } else {
+#pragma unroll
+          for (int i = 0; i < 16; ++i) o[i] = 0u;
+        }
+        if (dim < p.kv_rank) {
+#pragma unroll
+          for (int i = 0; i < 16; ++i) {
+            const int h = h0 + g + i;
+            if (h < p.heads) {
+              const float v = __uint_as_float(o[i]);
+              if (p.splits > 1) {
+                p.partial_o[((static_cast<int64_t>(b) * p.heads + h) * p.splits + split) * p.kv_rank + dim] = v;
+              } else {
+                const float l = s_l[g + i];
+                p.out[(static_cast<int64_t>(h) * p.rows_pad + b) * p.kv_rank + dim] = __float2bfloat16(l > 0.f ? v / l : 0.f);
+              }
+            }
+          }
+        }
+      }
+    }
+    if (!ok) {
+      // let copies that may still be in flight land before shared memory and TMEM are released
+      const uint64_t t0 = globaltimer_ns();
+      while (globaltimer_ns() - t0 < 200000ull) { __nanosleep(1000); }
+    }
+  }
+  __syncwarp();
+  tc_fence_before_sync();
+  __syncthreads();
+  if (warp == 0) {
+    tc_fence_after_sync();
+    tmem_dealloc(tmem_base, p.tmem_cols);
+  }
+}
+
+// One block per (head, sequence).
+__global__ void __launch_bounds__(128) latent_decode_merge_kernel(const float* __restrict__ po, const float* __restrict__ pml,
+                                                                  __nv_bfloat16* __restrict__ out, int64_t rows_pad,
+                                                                  int heads, int kv_rank, int splits) {
+  const int h = blockIdx.x, b = blockIdx.y;
+  const int64_t base = (static_cast<int64_t>(b) * heads + h) * splits;
+  float m = -1.0e29f;
+  for (int s = 0; s < splits; ++s) m = fmaxf(m, pml[(base + s) * 2]);
+  float l = 0.f;
+  for (int s = 0; s < splits; ++s) l += pml[(base + s) * 2 + 1] * exp2f(pml[(base + s) * 2] - m);
+  const float inv = l > 0.f ? 1.f / l : 0.f;
+  for (int d = threadIdx.x; d < kv_rank; d += 128) {
+    float v = 0.f;
+    for (int s = 0; s < splits; ++s) v += po[(base + s) * kv_rank + d] * exp2f(pml[(base + s) * 2] - m);
+    out[(static_cast<int64_t>(h) * rows_pad + b) * kv_rank + d] = __float2bfloat16(v * inv);
+  }
+}
+
+struct LatentDecodePlan {
+  int nh = 0, slabs = 0, slots = 0, ring = 0, chunks = 0, smem = 0;
+  uint32_t tmem_cols = 0;
+};
+
+// Heads per CTA, ring size and tensor-memory columns; nh == 0 when the sizes do not fit.
+inline LatentDecodePlan latent_decode_plan(int heads, int kv_rank, int row) {
+  LatentDecodePlan pl;
+  pl.slabs = (row + 63) / 64;
+  pl.chunks = (kv_rank + 127) / 128;
+  const int need = pl.slabs > 2 * pl.chunks ? pl.slabs : 2 * pl.chunks;
+  pl.slots = (need + 1) / 2 * 2;
+  for (int nh = heads > 32 ? 64 : (heads > 16 ? 32 : 16); nh >= 16; nh /= 2) {
+    const int cols = 128 + pl.chunks * nh;
+    if (cols > 512) continue;
+    const int fixed = 1024 + (pl.slabs + 2) * nh * 128;
+    int ring = (kLdSmemMax - fixed - kLdStatic) / kLdSlab / 2 * 2;
+    if (ring < 2 * pl.slots) continue;
+    const int small = 3 * pl.slots;                                 // three pages, if that lets two CTAs share an SM
+    if (ring > small && 2 * (fixed + small * kLdSlab + kLdStatic) <= kLdSmemMax && cols <= 256) ring = small;
+    if (ring > kLdBars * pl.slots) ring = kLdBars * pl.slots;
+    pl.nh = nh;
+    pl.ring = ring;
+    pl.smem = fixed + ring * kLdSlab;
+    pl.tmem_cols = 32;
+    while (pl.tmem_cols < static_cast<uint32_t>(cols)) pl.tmem_cols *= 2;
+    return pl;
+  }
+  return pl;
+}
+
+inline bool latent_decode_on_tensor_cores(const LatentDecodeArgs& a) {
+  const int row = a.kv_rank + a.rot_dim;
+  auto al16 = [](const void* p) { return (reinterpret_cast<uintptr_t>(p) & 15u) == 0; };
+  return a.dtype == 0 && a.block == kLdKeys && (row & 7) == 0 && a.kv_rank > 0 && a.scale > 0.f && al16(a.q) &&
+         al16(a.cache) && static_cast<int64_t>(a.num_blocks) * a.block < (1ll << 31) && a.splits <= 65535 &&
+         latent_decode_plan(a.heads, a.kv_rank, row).nh != 0;
+}
+
+template <int NH>
+int latent_decode_run(const LatentDecodeParams& p, dim3 grid, int smem, cudaStream_t stream) {
+  static PerDeviceInt configured;
+  if (configured.cur() < smem) {
+    const cudaError_t e =
+        cudaFuncSetAttribute(latent_decode_kernel<NH>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
+    if (e != cudaSuccess) return static_cast<int>(e);
+    configured.cur() = smem;
+  }
+  latent_decode_kernel<NH><<<grid, kLdThreads, smem, stream>>>(p);
+  return static_cast<int>(cudaGetLastError());
+}
+
+inline int launch_latent_decode_mma(const LatentDecodeArgs& a, cudaStream_t stream) {
+  const int row = a.kv_rank + a.rot_dim;
+  const LatentDecodePlan pl = latent_decode_plan(a.heads, a.kv_rank, row);
+  if (pl.nh == 0) return -60;
+  if (a.splits > 1 && (a.partial_o == nullptr || a.partial_ml == nullptr)) return -61;
+  LatentDecodeParams p;
+  const int64_t slots = static_cast<int64_t>(a.num_blocks) * a.block;
+  int r = make_tmap_2d(&p.tma_c, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, a.cache, static_cast<uint64_t>(row),
+                       static_cast<uint64_t>(slots), static_cast<uint64_t>(row), 64, kLdKeys);
+  if (r != 0) return -70 + r;
+  p.q = static_cast<const __nv_bfloat16*>(a.q); p.out = static_cast<__nv_bfloat16*>(a.out);
+  p.block_table = a.block_table; p.seq_lens = a.seq_lens;
+  p.partial_o = a.partial_o; p.partial_ml = a.partial_ml;
+  p.rows_pad = a.rows_pad;
+  p.heads = a.heads; p.kv_rank = a.kv_rank; p.row = row; p.max_blocks = a.max_blocks_per_seq; p.num_blocks = a.num_blocks;
+  p.window = a.window; p.splits = a.splits;
+  p.slabs = pl.slabs; p.slots = pl.slots; p.ring = pl.ring; p.chunks = pl.chunks; p.tmem_cols = pl.tmem_cols;
+  p.scale_log2 = a.scale * 1.4426950408889634f;
+  p.status = a.status;
+  dim3 grid(static_cast<unsigned>((a.heads + pl.nh - 1) / pl.nh), static_cast<unsigned>(a.batch),
+            static_cast<unsigned>(a.splits));
+  switch (pl.nh) {
+    case 16: r = latent_decode_run<16>(p, grid, pl.smem, stream); break;
+    case 32: r = latent_decode_run<32>(p, grid, pl.smem, stream); break;
+    default: r = latent_decode_run<64>(p, grid, pl.smem, stream); break;
+  }
+  if (r != 0 || a.splits == 1) return r;
+  latent_decode_merge_kernel<<<dim3(static_cast<unsigned>(a.heads), static_cast<unsigned>(a.batch)), 128, 0, stream>>>(
+      a.partial_o, a.partial_ml, p.out, a.rows_pad, a.heads, a.kv_rank, a.splits);
+  return static_cast<int>(cudaGetLastError());
+}
+
+}  // namespace yv

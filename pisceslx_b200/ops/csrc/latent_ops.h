@@ -105,7 +105,7 @@ struct LatentAttnArgs {
   uint32_t* status = nullptr;
 };
 int launch_latent_attn(const LatentAttnArgs& a, cudaStream_t stream);
-bool latent_attn_on_tensor_cores(const LatentAttnArgs& a);
+inline bool latent_attn_on_tensor_cores(const LatentAttnArgs& a);
 
 // One query token per batch row in the latent space.  q [heads, rows_pad, kv_rank + rot_dim] = [W_uk^T q | q rotated];
 // the weighted sum of the latents goes to out [heads, rows_pad, kv_rank].
@@ -124,7 +124,7 @@ struct LatentDecodeArgs {
   uint32_t* status = nullptr;
 };
 int launch_latent_decode(const LatentDecodeArgs& a, cudaStream_t stream);
-bool latent_decode_on_tensor_cores(const LatentDecodeArgs& a);
+inline bool latent_decode_on_tensor_cores(const LatentDecodeArgs& a);
 
 // out[t, h * vdim + j] = v[h, t, j] * sigmoid(gate[t, h])   (gate null: a plain transpose)
 int launch_head_gate(const void* v, int64_t v_hs, int64_t v_ts, const void* gate, int64_t gate_ld, void* out,

@@ -449,7 +449,7 @@ class PiscesLxBackendServer:
 
         from ..engine.loader import load_model_for_inference
         model = load_model_for_inference(getattr(self.args, "model_size", "0.01B"), getattr(self.args, "ckpt", None),
-                                         getattr(self.args, "device", None))
+                                         getattr(self.args, "device", None), getattr(self.args, "model_config", None))
         engine = YvInferenceEngine(model, cfg=YvEngineConfig(num_blocks=getattr(self.args, "kv_blocks", 1024)))
         app = PiscesLxInferService(engine, getattr(self.args, "model_size", "yv")).build_app()
         uvicorn.run(app, host=getattr(self.args, "host", "127.0.0.1"), port=int(getattr(self.args, "port", 8000)))

@@ -52,6 +52,13 @@ def visible(i, n, window):
     return [j for j in range(n) if j <= i and (window is None or i - j < window)]
 
 
+def attend(qn, qr, kn, kr, v, scale):
+    """One query position: qn [H, dim], qr [H, rot], keys kn [J, H, dim], kr [J, rot] (shared by the heads), values
+    v [J, H, vdim] -> [H, vdim]."""
+    s = (torch.einsum("hd,jhd->hj", qn, kn) + torch.einsum("hd,jd->hj", qr, kr)) * scale
+    return torch.einsum("hj,jhd->hd", torch.softmax(s, -1), v)
+
+
 def latent_attention(h, W, p, mx, eps):
     """h [T, width] (normed input, positions 0..T-1) -> [T, width]."""
     T = h.shape[0]
@@ -69,9 +76,8 @@ def latent_attention(h, W, p, mx, eps):
     for t in range(T):
         js = visible(t, T, window)
         lo, hi = js[0], js[-1] + 1                       # the visible keys are one run
-        qn, qr = q[t, :, :dim], rotate(q[t, :, dim:], t, mx["rot"])
-        s = (torch.einsum("hd,jhd->hj", qn, kn[lo:hi]) + torch.einsum("hd,jd->hj", qr, kr[lo:hi])) * mx["scale"]
-        out[t] = torch.einsum("hj,jhd->hd", torch.softmax(s, -1), v[lo:hi]) * gate[t][:, None]
+        out[t] = attend(q[t, :, :dim], rotate(q[t, :, dim:], t, mx["rot"]), kn[lo:hi], kr[lo:hi], v[lo:hi],
+                        mx["scale"]) * gate[t][:, None]
     return out.reshape(T, H * vd) @ W[p + "o"].T
 
 
