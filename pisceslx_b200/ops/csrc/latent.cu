@@ -49,9 +49,102 @@ __device__ __forceinline__ int table_row(const int* positions, int64_t t, int ma
   return pos;
 }
 
+// Four consecutive elements (8 bytes of bf16, 16 of fp32).
+__device__ __forceinline__ void load4(const float* p, float (&f)[4]) {
+  const float4 t = *reinterpret_cast<const float4*>(p);
+  f[0] = t.x; f[1] = t.y; f[2] = t.z; f[3] = t.w;
+}
+__device__ __forceinline__ void load4(const __nv_bfloat16* p, float (&f)[4]) {
+  const uint2 t = *reinterpret_cast<const uint2*>(p);
+  f[0] = __uint_as_float(t.x << 16); f[1] = __uint_as_float(t.x & 0xFFFF0000u);
+  f[2] = __uint_as_float(t.y << 16); f[3] = __uint_as_float(t.y & 0xFFFF0000u);
+}
+__device__ __forceinline__ void store4(float* p, const float (&f)[4]) {
+  *reinterpret_cast<float4*>(p) = make_float4(f[0], f[1], f[2], f[3]);
+}
+__device__ __forceinline__ void store4(__nv_bfloat16* p, const float (&f)[4]) {
+  *reinterpret_cast<uint2*>(p) = make_uint2(pack_bf16(f[0], f[1]), pack_bf16(f[2], f[3]));
+}
 constexpr int kPrepThreads = 128;
+constexpr int kPrepVecs = 4;           // groups of four per thread and latent kept in registers
 
-// One block per token.
+// One block per token, both latents in registers (ranks up to 2048, all sizes and pitches multiples of 8).
+template <typename T>
+__global__ void __launch_bounds__(kPrepThreads) latent_prep_vec_kernel(const LatentPrepArgs p) {
+  __shared__ float red[2][kPrepThreads / 32];
+  const int64_t t = blockIdx.x;
+  const T* in = static_cast<const T*>(p.in) + t * p.ld;
+  const T* kv = in + p.q_rank;
+  const int nq = p.q_rank >> 2, nk = p.kv_rank >> 2;
+  float q[kPrepVecs][4], k[kPrepVecs][4];
+  float sq = 0.f, sk = 0.f;
+#pragma unroll
+  for (int i = 0; i < kPrepVecs; ++i) {
+    const int c = threadIdx.x + i * kPrepThreads;
+#pragma unroll
+    for (int j = 0; j < 4; ++j) q[i][j] = k[i][j] = 0.f;
+    if (c < nq) load4(in + c * 4, q[i]);
+    if (c < nk) load4(kv + c * 4, k[i]);
+  }
+#pragma unroll
+  for (int i = 0; i < kPrepVecs; ++i)
+#pragma unroll
+    for (int j = 0; j < 4; ++j) { sq += q[i][j] * q[i][j]; sk += k[i][j] * k[i][j]; }
+  sq = warp_sum(sq);
+  sk = warp_sum(sk);
+  if ((threadIdx.x & 31) == 0) { red[0][threadIdx.x >> 5] = sq; red[1][threadIdx.x >> 5] = sk; }
+  __syncthreads();
+  sq = sk = 0.f;
+#pragma unroll
+  for (int i = 0; i < kPrepThreads / 32; ++i) { sq += red[0][i]; sk += red[1][i]; }
+  const float rq = 1.f / sqrtf(sq / static_cast<float>(p.q_rank) + p.eps);
+  const float rk = 1.f / sqrtf(sk / static_cast<float>(p.kv_rank) + p.eps);
+  const int row = p.kv_rank + p.rot_dim;
+  T* out_rows = p.rows != nullptr ? static_cast<T*>(p.rows) + t * row : nullptr;
+  T* out_cache = nullptr;
+  if (p.cache != nullptr) {
+    const int64_t slot = p.slot_map[t];
+    if (slot >= p.num_slots) { if (threadIdx.x == 0) report(p.status, kStatusIndexOutOfRange); }
+    else if (slot >= 0) out_cache = static_cast<T*>(p.cache) + slot * row;
+  }
+  auto put = [&](int i, const float (&f)[4]) {
+    if (out_rows != nullptr) store4(out_rows + i, f);
+    if (out_cache != nullptr) store4(out_cache + i, f);
+  };
+  T* cq = static_cast<T*>(p.cq) + t * p.cq_ld;
+#pragma unroll
+  for (int i = 0; i < kPrepVecs; ++i) {
+    const int c = threadIdx.x + i * kPrepThreads;
+    float w[4];
+    if (c < nq) {
+      load4(static_cast<const T*>(p.w_q) + c * 4, w);
+#pragma unroll
+      for (int j = 0; j < 4; ++j) q[i][j] *= rq * w[j];
+      store4(cq + c * 4, q[i]);
+    }
+    if (c < nk) {
+      load4(static_cast<const T*>(p.w_kv) + c * 4, w);
+#pragma unroll
+      for (int j = 0; j < 4; ++j) k[i][j] *= rk * w[j];
+      put(c * 4, k[i]);
+    }
+  }
+  const int half = p.rot_dim >> 1;
+  const int64_t pos = table_row(p.positions, t, p.max_pos, p.status);
+  for (int i = threadIdx.x * 4; i < half; i += kPrepThreads * 4) {
+    float c[4], s[4], u[4], v[4], a[4], b[4];
+    load4(p.cos_t + pos * half + i, c);
+    load4(p.sin_t + pos * half + i, s);
+    load4(kv + p.kv_rank + i, u);
+    load4(kv + p.kv_rank + half + i, v);
+#pragma unroll
+    for (int j = 0; j < 4; ++j) { a[j] = u[j] * c[j] - v[j] * s[j]; b[j] = v[j] * c[j] + u[j] * s[j]; }
+    put(p.kv_rank + i, a);
+    put(p.kv_rank + half + i, b);
+  }
+}
+
+// One block per token, any sizes.
 template <typename T>
 __global__ void __launch_bounds__(kPrepThreads) latent_prep_kernel(const LatentPrepArgs p) {
   __shared__ float red[2][kPrepThreads / 32];
@@ -98,45 +191,69 @@ __global__ void __launch_bounds__(kPrepThreads) latent_prep_kernel(const LatentP
   }
 }
 
-template <typename T>
+// Work items of N consecutive elements (4 or 1): all rotary pairs of all tokens, then all plain parts.
+template <typename T, int N>
 __global__ void __launch_bounds__(256) latent_query_kernel(const LatentQueryArgs p) {
-  const int64_t t = blockIdx.x;
-  const int half = p.rot_dim >> 1;
-  const int hd = p.dim + p.rot_dim;
-  const T* q = static_cast<const T*>(p.q) + t * p.ld;
-  const int64_t pos = table_row(p.positions, t, p.max_pos, p.status);
-  for (int i = threadIdx.x; i < p.heads * half; i += 256) {
-    const int h = i / half, j = i - h * half;
-    const float c = p.cos_t[pos * half + j], s = p.sin_t[pos * half + j];
-    const T* src = q + h * hd + p.dim;
-    const float u = to_f(src[j]), v = to_f(src[half + j]);
-    T* dst = static_cast<T*>(p.rope_out) + h * p.rope_hs + t * p.rope_ts;
-    dst[j] = from_f<T>(u * c - v * s);                 // in place: a pair is read and written by one thread
-    dst[half + j] = from_f<T>(v * c + u * s);
-  }
-  if (p.nope_out != nullptr)
-    for (int i = threadIdx.x; i < p.heads * p.dim; i += 256) {
-      const int h = i / p.dim, j = i - h * p.dim;
-      (static_cast<T*>(p.nope_out) + h * p.nope_hs + t * p.nope_ts)[j] = q[h * hd + j];
+  const int half = p.rot_dim >> 1, hv = half / N, dv = p.nope_out != nullptr ? p.dim / N : 0;
+  const int per_head = hv + dv, hd = p.dim + p.rot_dim;
+  const int64_t i = static_cast<int64_t>(blockIdx.x) * 256 + threadIdx.x;
+  const int64_t th = i / per_head;
+  const int e = static_cast<int>(i - th * per_head);
+  const int64_t t = th / p.heads;
+  const int h = static_cast<int>(th - t * p.heads);
+  if (t >= p.T) return;
+  const T* q = static_cast<const T*>(p.q) + t * p.ld + static_cast<int64_t>(h) * hd;
+  if (e < hv) {
+    int pos = p.positions[t];
+    if (pos < 0 || pos >= p.max_pos) {
+      report(p.status, kStatusIndexOutOfRange);
+      pos = pos < 0 ? 0 : p.max_pos - 1;
     }
+    const int j = e * N;
+    const float* ct = p.cos_t + static_cast<int64_t>(pos) * half + j;
+    const float* st = p.sin_t + static_cast<int64_t>(pos) * half + j;
+    const T* src = q + p.dim + j;
+    T* dst = static_cast<T*>(p.rope_out) + h * p.rope_hs + t * p.rope_ts + j;   // in place: one thread owns a pair
+    if constexpr (N == 4) {
+      float c[4], s[4], u[4], v[4], a[4], b[4];
+      load4(ct, c); load4(st, s); load4(src, u); load4(src + half, v);
+#pragma unroll
+      for (int k = 0; k < 4; ++k) { a[k] = u[k] * c[k] - v[k] * s[k]; b[k] = v[k] * c[k] + u[k] * s[k]; }
+      store4(dst, a);
+      store4(dst + half, b);
+    } else {
+      const float u = to_f(src[0]), v = to_f(src[half]);
+      dst[0] = from_f<T>(u * ct[0] - v * st[0]);
+      dst[half] = from_f<T>(v * ct[0] + u * st[0]);
+    }
+  } else {
+    const int j = (e - hv) * N;
+    T* dst = static_cast<T*>(p.nope_out) + h * p.nope_hs + t * p.nope_ts + j;
+    if constexpr (N == 4) { float f[4]; load4(q + j, f); store4(dst, f); }
+    else dst[0] = q[j];
+  }
 }
 
+// One warp per row.
 template <typename T>
-__global__ void __launch_bounds__(128) latent_gather_kernel(const T* __restrict__ cache, int64_t num_slots,
-                                                            const int* __restrict__ slots, T* __restrict__ out, int row,
-                                                            uint32_t* status) {
-  const int64_t i = blockIdx.x;
+__global__ void __launch_bounds__(256) latent_gather_kernel(const T* __restrict__ cache, int64_t num_slots,
+                                                            const int* __restrict__ slots, T* __restrict__ out, int64_t n,
+                                                            int row, uint32_t* status) {
+  const int64_t i = static_cast<int64_t>(blockIdx.x) * 8 + (threadIdx.x >> 5);
+  const int lane = threadIdx.x & 31;
+  if (i >= n) return;
   const int64_t s = slots[i];
   const bool ok = s >= 0 && s < num_slots;
-  if (!ok && threadIdx.x == 0) report(status, kStatusIndexOutOfRange);
+  if (!ok && lane == 0) report(status, kStatusIndexOutOfRange);
   const T* src = cache + (ok ? s : 0) * row;
   T* dst = out + i * row;
   if ((row * sizeof(T)) % 16 == 0) {
     const int nv = static_cast<int>(row * sizeof(T) / 16);
-    for (int c = threadIdx.x; c < nv; c += 128)
+#pragma unroll 4
+    for (int c = lane; c < nv; c += 32)
       reinterpret_cast<uint4*>(dst)[c] = ok ? reinterpret_cast<const uint4*>(src)[c] : make_uint4(0, 0, 0, 0);
   } else {
-    for (int c = threadIdx.x; c < row; c += 128) dst[c] = ok ? src[c] : from_f<T>(0.f);
+    for (int c = lane; c < row; c += 32) dst[c] = ok ? src[c] : from_f<T>(0.f);
   }
 }
 
@@ -305,7 +422,14 @@ int launch_latent_prep(const LatentPrepArgs& a, cudaStream_t stream) {
   if (a.ld < a.q_rank + a.kv_rank + a.rot_dim || a.cq_ld < a.q_rank) return -2;
   if (a.cache != nullptr && a.slot_map == nullptr) return -3;
   const unsigned grid = static_cast<unsigned>(a.T);
-  if (a.dtype == 1) latent_prep_kernel<float><<<grid, kPrepThreads, 0, stream>>>(a);
+  const int esz = a.dtype == 1 ? 4 : 2;
+  auto al = [&](const void* p) { return (reinterpret_cast<uintptr_t>(p) % (4 * esz)) == 0; };
+  const bool vec = ((a.q_rank | a.kv_rank | a.rot_dim) & 7) == 0 && ((a.ld | a.cq_ld) & 3) == 0 &&
+                   a.q_rank <= 4 * kPrepVecs * kPrepThreads && a.kv_rank <= 4 * kPrepVecs * kPrepThreads && al(a.in) &&
+                   al(a.cq) && al(a.rows) && al(a.cache) && al(a.w_q) && al(a.w_kv);
+  if (vec && a.dtype == 1) latent_prep_vec_kernel<float><<<grid, kPrepThreads, 0, stream>>>(a);
+  else if (vec) latent_prep_vec_kernel<__nv_bfloat16><<<grid, kPrepThreads, 0, stream>>>(a);
+  else if (a.dtype == 1) latent_prep_kernel<float><<<grid, kPrepThreads, 0, stream>>>(a);
   else latent_prep_kernel<__nv_bfloat16><<<grid, kPrepThreads, 0, stream>>>(a);
   return static_cast<int>(cudaGetLastError());
 }
@@ -313,22 +437,33 @@ int launch_latent_prep(const LatentPrepArgs& a, cudaStream_t stream) {
 int launch_latent_query(const LatentQueryArgs& a, cudaStream_t stream) {
   if (a.T <= 0) return 0;
   if (a.heads <= 0 || a.dim < 0 || a.rot_dim <= 0 || (a.rot_dim & 1) || a.max_pos <= 0) return -1;
-  const unsigned grid = static_cast<unsigned>(a.T);
-  if (a.dtype == 1) latent_query_kernel<float><<<grid, 256, 0, stream>>>(a);
-  else latent_query_kernel<__nv_bfloat16><<<grid, 256, 0, stream>>>(a);
+  const int esz = a.dtype == 1 ? 4 : 2;
+  auto al = [&](const void* p) { return (reinterpret_cast<uintptr_t>(p) % (4 * esz)) == 0; };
+  const bool vec = ((a.dim | (a.rot_dim >> 1)) & 3) == 0 && ((a.ld | a.nope_hs | a.nope_ts | a.rope_hs | a.rope_ts) & 3) == 0 &&
+                   al(a.q) && al(a.nope_out) && al(a.rope_out);
+  const int n = vec ? 4 : 1;
+  const int64_t items = a.T * a.heads * ((a.rot_dim >> 1) / n + (a.nope_out != nullptr ? a.dim / n : 0));
+  const unsigned grid = static_cast<unsigned>((items + 255) / 256);
+  if (a.dtype == 1) {
+    if (vec) latent_query_kernel<float, 4><<<grid, 256, 0, stream>>>(a);
+    else latent_query_kernel<float, 1><<<grid, 256, 0, stream>>>(a);
+  } else {
+    if (vec) latent_query_kernel<__nv_bfloat16, 4><<<grid, 256, 0, stream>>>(a);
+    else latent_query_kernel<__nv_bfloat16, 1><<<grid, 256, 0, stream>>>(a);
+  }
   return static_cast<int>(cudaGetLastError());
 }
 
 int launch_latent_gather(const void* cache, int64_t num_slots, const int* slots, void* out, int64_t n, int row,
                          int dtype, uint32_t* status, cudaStream_t stream) {
   if (n <= 0) return 0;
-  const unsigned grid = static_cast<unsigned>(n);
+  const unsigned grid = static_cast<unsigned>((n + 7) / 8);
   if (dtype == 1)
-    latent_gather_kernel<float><<<grid, 128, 0, stream>>>(static_cast<const float*>(cache), num_slots, slots,
-                                                          static_cast<float*>(out), row, status);
+    latent_gather_kernel<float><<<grid, 256, 0, stream>>>(static_cast<const float*>(cache), num_slots, slots,
+                                                          static_cast<float*>(out), n, row, status);
   else
-    latent_gather_kernel<__nv_bfloat16><<<grid, 128, 0, stream>>>(static_cast<const __nv_bfloat16*>(cache), num_slots,
-                                                                  slots, static_cast<__nv_bfloat16*>(out), row, status);
+    latent_gather_kernel<__nv_bfloat16><<<grid, 256, 0, stream>>>(static_cast<const __nv_bfloat16*>(cache), num_slots,
+                                                                  slots, static_cast<__nv_bfloat16*>(out), n, row, status);
   return static_cast<int>(cudaGetLastError());
 }
 

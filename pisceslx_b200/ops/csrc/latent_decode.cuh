@@ -8,10 +8,11 @@
 // The M dimension of the first product reads past the NH real rows of Q into whatever follows in shared memory; those
 // lanes of S are never read.
 //
-// grid = (head groups of NH, sequences, key ranges), 160 threads:
+// grid = (head groups of NH, sequences, key ranges), 192 threads:
 //   warps 0..3  softmax: thread t owns head t (TMEM lane t of S, no cross-lane reductions); O^T is rescaled by all
 //               128 threads (lane = latent dimension) when a head's reference maximum moves, which is rare
-//   warp 4      one lane issues the TMA copies and both products
+//   warp 4      one lane issues both products; a page that has arrived is scored before the product of the page in front
+//   warp 5      one lane issues the TMA copies
 // The page slabs travel through a ring counted in slabs, so that a part of the page after next is already in flight
 // when two whole pages do not leave room for a third.  A page takes an even number of ring slots: the pair of slabs
 // behind one 128-row product is always contiguous.
@@ -40,7 +41,7 @@ struct LatentDecodeParams {
   uint32_t* status;
 };
 
-constexpr int kLdThreads = 160;
+constexpr int kLdThreads = 192;
 constexpr int kLdKeys = 64;
 constexpr int kLdSlab = kLdKeys * 128;
 constexpr int kLdBars = 4;                                  // pages whose arrival can be tracked at a time
@@ -82,7 +83,7 @@ __global__ void __launch_bounds__(kLdThreads) latent_decode_kernel(const __grid_
   uint8_t* sQ = sm;                                         // [slabs][NH][128 B]
   uint8_t* sP = sQ + p.slabs * kQSlab;                      // [2][NH][128 B]
   uint8_t* ring = sP + 2 * kQSlab;                          // [ring][64 keys][128 B]
-  __shared__ uint64_t full_bar[kLdBars], s_bar[2], pv_bar[2], p_bar[2];
+  __shared__ uint64_t full_bar[kLdBars], empty_bar[kLdBars], s_bar[2], pv_bar[2], p_bar[2];
   __shared__ uint32_t tmem_slot;
   __shared__ float s_alpha[2][NH], s_l[NH];
   __shared__ int s_table[kLdTableCap];
@@ -110,7 +111,7 @@ __global__ void __launch_bounds__(kLdThreads) latent_decode_kernel(const __grid_
 
   if (tid == 0) {
     tma_prefetch_desc(&p.tma_c);
-    for (int i = 0; i < kLdBars; ++i) mbar_init(&full_bar[i], 1);
+    for (int i = 0; i < kLdBars; ++i) { mbar_init(&full_bar[i], 1); mbar_init(&empty_bar[i], 1); }
     for (int i = 0; i < 2; ++i) { mbar_init(&s_bar[i], 1); mbar_init(&pv_bar[i], 1); mbar_init(&p_bar[i], 128); }
     fence_barrier_init();
   }
@@ -134,73 +135,92 @@ __global__ void __launch_bounds__(kLdThreads) latent_decode_kernel(const __grid_
   const uint32_t tmem_base = tmem_slot;
   const uint32_t tO = tmem_base + 128u;                     // S buffers at columns 0 and 64
 
-  if (warp == 4) {
-    // ------------------------------------ issuer ---------------------------------------------
-    if (lane == 0 && n_tiles > 0) {
-      int next = 0;                                         // next ring slot (counted from the first page on) to fill
-      auto fill = [&](int pages_done) {
-        const int limit = min(pages_done * p.slots + p.ring, n_tiles * p.slots);
-        for (; next < limit; ++next) {
-          const int j = next / p.slots, c = next - j * p.slots;
-          // a page of arrivals is tracked by barrier j % kLdBars: its previous user must have been consumed
-          if (j >= pages_done + kLdBars) break;
-          if (c == 0) mbar_expect_tx(&full_bar[j % kLdBars], static_cast<uint32_t>(p.slabs) * kLdSlab);
-          if (c >= p.slabs) continue;
-          int page = table[j];
-          if (page < 0 || page >= p.num_blocks) {           // reported; its keys are masked by the softmax warps
-            if (p.status != nullptr) atomicOr(p.status, kStatusIndexOutOfRange);
-            page = 0;
-          }
-          tma_load_2d(ring + static_cast<size_t>(next % p.ring) * kLdSlab, &p.tma_c, &full_bar[j % kLdBars], c * 64,
-                      page * kLdKeys);
+  if (warp == 5) {
+    // ------------------------------------ TMA producer ---------------------------------------
+    if (lane == 0) {
+      bool ok = true;
+      int slot = 0;                                         // ring slot of the next slab
+      int room = p.ring;                                    // free ring slots
+      int freed = 0;                                        // pages known to have been consumed
+      for (int j = 0; j < n_tiles && ok; ++j) {
+        // the barrier of page j was last used by page j - kLdBars
+        while (ok && freed + kLdBars <= j) {
+          ok = mbar_wait(&empty_bar[freed % kLdBars], (freed / kLdBars) & 1u, p.status);
+          ++freed;
+          room += p.slots;
         }
-      };
-      const int steps = (p.row + 15) / 16;
-      const uint32_t aQ = smem_u32(sQ), aR = smem_u32(ring), aP = smem_u32(sP);
-      auto slab_addr = [&](int j, int c) { return aR + static_cast<uint32_t>((j * p.slots + c) % p.ring) * kLdSlab; };
+        if (!ok) break;
+        uint64_t* full = &full_bar[j % kLdBars];
+        mbar_expect_tx(full, static_cast<uint32_t>(p.slabs) * kLdSlab);
+        int page = table[j];
+        if (page < 0 || page >= p.num_blocks) {             // reported; its keys are masked by the softmax warps
+          if (p.status != nullptr) atomicOr(p.status, kStatusIndexOutOfRange);
+          page = 0;
+        }
+        for (int c = 0; c < p.slots && ok; ++c) {
+          while (ok && room == 0) {
+            ok = mbar_wait(&empty_bar[freed % kLdBars], (freed / kLdBars) & 1u, p.status);
+            ++freed;
+            room += p.slots;
+          }
+          if (!ok) break;
+          if (c < p.slabs) tma_load_2d(ring + static_cast<size_t>(slot) * kLdSlab, &p.tma_c, full, c * 64, page * kLdKeys);
+          --room;
+          if (++slot == p.ring) slot = 0;
+        }
+      }
+    }
+  } else if (warp == 4) {
+    // ------------------------------------ MMA issuer -----------------------------------------
+    if (lane == 0 && n_tiles > 0) {
+      // descriptors differ in their address field only: base + byte offset / 16
+      const uint64_t dQ = make_smem_desc(smem_u32(sQ), 16, 1024), dR = make_smem_desc(smem_u32(ring), 16, 1024);
+      const uint64_t dC = make_smem_desc(smem_u32(ring), kLdSlab, 1024), dP = make_smem_desc(smem_u32(sP), 16, 1024);
+      int qk_slot = 0, pv_slot = 0;                         // ring slots of the next page to score / to accumulate
       auto issue_qk = [&](int j) -> bool {
         if (!mbar_wait(&full_bar[j % kLdBars], (j / kLdBars) & 1u, p.status)) return false;
         tc_fence_after_sync();
         const uint32_t dS = tmem_base + static_cast<uint32_t>((j & 1) * 64);
-        for (int kk = 0; kk < steps; ++kk) {
-          const int c = kk >> 2, o = (kk & 3) * 32;
-          tc_mma_f16_ss(dS, make_smem_desc(aQ + c * kQSlab + o, 16, 1024), make_smem_desc(slab_addr(j, c) + o, 16, 1024),
-                        kIdescQK, kk != 0 ? 1u : 0u);
+        int slot = qk_slot;
+        for (int c = 0; c < p.slabs; ++c) {                 // columns past the row are zero in both operands
+          const uint64_t a = dQ + static_cast<uint64_t>(c * (kQSlab >> 4)), k = dR + static_cast<uint64_t>(slot * (kLdSlab >> 4));
+#pragma unroll
+          for (int kk = 0; kk < 4; ++kk) tc_mma_f16_ss(dS, a + kk * 2, k + kk * 2, kIdescQK, (c | kk) != 0 ? 1u : 0u);
+          if (++slot == p.ring) slot = 0;
         }
+        qk_slot += p.slots;
+        if (qk_slot >= p.ring) qk_slot -= p.ring;
         tc_commit(&s_bar[j & 1]);
         return true;
       };
-      fill(0);
       bool ok = issue_qk(0);
       for (int j = 0; j < n_tiles && ok; ++j) {
         bool ahead = j + 1 >= n_tiles;
-        if (!ahead && next >= (j + 1) * p.slots + p.slabs) {      // the next page is on its way: score it now
-          ok = issue_qk(j + 1);
+        if (!ahead && mbar_test_wait(&full_bar[(j + 1) % kLdBars], ((j + 1) / kLdBars) & 1u)) {
+          ok = issue_qk(j + 1);                             // the next page is here: score it under this page's softmax
           ahead = true;
-          if (!ok) break;
-        }
-        if (j > 0) {
-          ok = mbar_wait(&pv_bar[(j - 1) & 1], ((j - 1) >> 1) & 1u, p.status);
-          if (!ok) break;
-          fill(j);                                                // pages 0 .. j - 1 have been consumed
-        }
-        if (!ahead) {
-          ok = issue_qk(j + 1);
           if (!ok) break;
         }
         // (one barrier per P buffer: the softmax warps may finish page j + 1 before this thread looks at page j)
         ok = mbar_wait(&p_bar[j & 1], (j >> 1) & 1u, p.status);
         if (!ok) break;
         tc_fence_after_sync();
-        const uint32_t bP = aP + static_cast<uint32_t>((j & 1) * kQSlab);
+        const uint64_t bP = dP + static_cast<uint64_t>((j & 1) * (kQSlab >> 4));
+        int slot = pv_slot;
         for (int m = 0; m < p.chunks; ++m) {
-          const uint32_t aC = slab_addr(j, 2 * m);
+          const uint64_t aC = dC + static_cast<uint64_t>(slot * (kLdSlab >> 4));
 #pragma unroll
           for (int kk = 0; kk < kLdKeys / 16; ++kk)
-            tc_mma_f16_ss(tO + static_cast<uint32_t>(m * NH), make_smem_desc(aC + kk * 2048, kLdSlab, 1024),
-                          make_smem_desc(bP + kk * 32, 16, 1024), kIdescPV, (j | kk) != 0 ? 1u : 0u);
+            tc_mma_f16_ss(tO + static_cast<uint32_t>(m * NH), aC + kk * (2048 >> 4), bP + kk * 2, kIdescPV,
+                          (j | kk) != 0 ? 1u : 0u);
+          slot += 2;
+          if (slot >= p.ring) slot -= p.ring;
         }
+        pv_slot += p.slots;
+        if (pv_slot >= p.ring) pv_slot -= p.ring;
         tc_commit(&pv_bar[j & 1]);
+        tc_commit(&empty_bar[j % kLdBars]);
+        if (!ahead) ok = issue_qk(j + 1);
       }
     }
   } else {

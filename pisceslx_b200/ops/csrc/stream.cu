@@ -181,15 +181,24 @@ __device__ __forceinline__ float gelu_tanh(float z) {
 
 template <typename T>
 __global__ void __launch_bounds__(256) gelu_kernel(const T* __restrict__ in, T* __restrict__ out, int64_t n) {
-  const int64_t i = (static_cast<int64_t>(blockIdx.x) * 256 + threadIdx.x) * 4;
-  if (i + 4 <= n) {
-    float f[4];
-    load4(in + i, f);
+  // four groups of four per thread, all loads before the arithmetic
+  const int64_t i0 = static_cast<int64_t>(blockIdx.x) * 4096 + threadIdx.x * 4;
+  float f[4][4];
 #pragma unroll
-    for (int j = 0; j < 4; ++j) f[j] = gelu_erf(f[j]);
-    store4(out + i, f);
-  } else {
-    for (int64_t j = i; j < n; ++j) out[j] = from_f<T>(gelu_erf(to_f(in[j])));
+  for (int u = 0; u < 4; ++u) {
+    const int64_t i = i0 + u * 1024;
+    if (i + 4 <= n) load4(in + i, f[u]);
+  }
+#pragma unroll
+  for (int u = 0; u < 4; ++u) {
+    const int64_t i = i0 + u * 1024;
+    if (i + 4 <= n) {
+#pragma unroll
+      for (int j = 0; j < 4; ++j) f[u][j] = gelu_erf(f[u][j]);
+      store4(out + i, f[u]);
+    } else {
+      for (int64_t j = i; j < n; ++j) out[j] = from_f<T>(gelu_erf(to_f(in[j])));
+    }
   }
 }
 
@@ -266,7 +275,7 @@ int launch_stream_norm(const StreamNormArgs& a, cudaStream_t stream) {
 int launch_gelu(const void* in, void* out, int64_t n, int dtype, cudaStream_t stream) {
   if (n <= 0) return 0;
   if ((reinterpret_cast<uintptr_t>(in) & 15u) != 0 || (reinterpret_cast<uintptr_t>(out) & 15u) != 0) return -1;
-  const unsigned grid = static_cast<unsigned>((n + 1023) / 1024);
+  const unsigned grid = static_cast<unsigned>((n + 4095) / 4096);
   if (dtype == 1) gelu_kernel<float><<<grid, 256, 0, stream>>>(static_cast<const float*>(in), static_cast<float*>(out), n);
   else gelu_kernel<__nv_bfloat16><<<grid, 256, 0, stream>>>(static_cast<const __nv_bfloat16*>(in),
                                                             static_cast<__nv_bfloat16*>(out), n);

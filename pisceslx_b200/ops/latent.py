@@ -181,12 +181,14 @@ def latent_attention(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, kr: torc
     return o
 
 
-def decode_splits(batch: int, heads: int, table_width: int, block: int, window: Optional[int]) -> int:
+def decode_splits(batch: int, heads: int, table_width: int, block: int, window: Optional[int], row: int = 576) -> int:
     """Key ranges per sequence of the latent decode kernel.  It depends on shapes only (so that a captured step can be
-    replayed): two CTAs per SM's worth of ranges, none shorter than four pages."""
+    replayed): the count that minimises the waves of CTAs times the pages of one CTA, with two pages' time for a CTA's
+    start and end.  A small row lets two CTAs share an SM."""
     pages = table_width if not window else min(table_width, -(-window // block) + 1)
-    ctas = batch * -(-heads // 64)
-    return max(1, min(32, -(-296 // max(ctas, 1)), pages // 4))
+    ctas, room = batch * -(-heads // 64), 148 * (2 if row <= 192 else 1)
+    best = min(range(1, min(32, max(pages, 1)) + 1), key=lambda s: (-(-ctas * s // room) * (-(-pages // s) + 2), s))
+    return best
 
 
 def latent_decode(q_lat: torch.Tensor, cache: torch.Tensor, kv_rank: int, block_table: torch.Tensor,
@@ -200,7 +202,7 @@ def latent_decode(q_lat: torch.Tensor, cache: torch.Tensor, kv_rank: int, block_
         return ref.latent_decode(q_lat, cache, kv_rank, block_table, seq_lens, window, scale)
     out = torch.empty(heads, R, kv_rank, dtype=q_lat.dtype, device=q_lat.device)
     if splits <= 0:
-        splits = decode_splits(B, heads, block_table.shape[1], cache.shape[1], window)
+        splits = decode_splits(B, heads, block_table.shape[1], cache.shape[1], window, cache.shape[2])
     po = pml = None
     if splits > 1:
         po = torch.empty(B * heads * splits * kv_rank, dtype=torch.float32, device=q_lat.device)
