@@ -8,11 +8,15 @@
 // The M dimension of the first product reads past the NH real rows of Q into whatever follows in shared memory; those
 // lanes of S are never read.
 //
-// grid = (head groups of NH, sequences, key ranges), 192 threads:
-//   warps 0..3  softmax: thread t owns head t (TMEM lane t of S, no cross-lane reductions); O^T is rescaled by all
-//               128 threads (lane = latent dimension) when a head's reference maximum moves, which is rare
-//   warp 4      one lane issues both products; a page that has arrived is scored before the product of the page in front
-//   warp 5      one lane issues the TMA copies
+// grid = (head groups of NH, sequences, key ranges), 288 threads.  A warp reads the 32 TMEM lanes of its index modulo
+// four, so two warps share the scores of the same heads, half a page each:
+//   scoring     warps with (index % 4) < NH / 32: thread = (head, half of the page); both threads of a head keep the
+//               same reference maximum, which moves only when a score exceeds it by 2^8 (one flag per page, agreed at
+//               the barrier; the exchange of maxima and the rescaling of O^T are a rare path)
+//   rescaling   warps 0..3 (lane = latent dimension), also the final output
+//   warps 6, 8  one lane each issues the first and the second product.  The products are short, so issuing them is a
+//               part of the page's time that is worth sharing; scores run up to two pages ahead
+//   warp 7      one lane issues the TMA copies
 // The page slabs travel through a ring counted in slabs, so that a part of the page after next is already in flight
 // when two whole pages do not leave room for a third.  A page takes an even number of ring slots: the pair of slabs
 // behind one 128-row product is always contiguous.
@@ -41,7 +45,7 @@ struct LatentDecodeParams {
   uint32_t* status;
 };
 
-constexpr int kLdThreads = 192;
+constexpr int kLdThreads = 288;
 constexpr int kLdKeys = 64;
 constexpr int kLdSlab = kLdKeys * 128;
 constexpr int kLdBars = 4;                                  // pages whose arrival can be tracked at a time
@@ -49,8 +53,9 @@ constexpr int kLdSmemMax = 227 * 1024;
 constexpr int kLdTableCap = 512;                            // block-table entries of a key range staged in shared memory
 constexpr int kLdStatic = 4096;                             // bound on the kernel's static shared memory
 
-// Barrier over the 128 softmax threads with an OR of `v`.  The instruction is warp-aligned: lanes that left a bounded
-// wait at different times are brought together first.
+// Barrier over the scoring and rescaling threads (COUNT of them) with an OR of `v`.  The instruction is warp-aligned:
+// lanes that left a bounded wait at different times are brought together first.
+template <int COUNT>
 __device__ __forceinline__ bool ld_barrier_or(bool v) {
   uint32_t r;
   __syncwarp();
@@ -58,11 +63,11 @@ __device__ __forceinline__ bool ld_barrier_or(bool v) {
       "{\n"
       ".reg .pred pin, pout;\n"
       "setp.ne.u32 pin, %1, 0;\n"
-      "bar.red.or.pred pout, 1, 128, pin;\n"
+      "bar.red.or.pred pout, 1, %2, pin;\n"
       "selp.u32 %0, 1, 0, pout;\n"
       "}\n"
       : "=r"(r)
-      : "r"(static_cast<uint32_t>(v))
+      : "r"(static_cast<uint32_t>(v)), "n"(COUNT)
       : "memory");
   return r != 0u;
 }
@@ -74,9 +79,11 @@ __device__ __forceinline__ float ld_exp2(float x) {
 }
 
 template <int NH>
-__global__ void __launch_bounds__(kLdThreads) latent_decode_kernel(const __grid_constant__ LatentDecodeParams p) {
+__global__ void __launch_bounds__(kLdThreads, 2) latent_decode_kernel(const __grid_constant__ LatentDecodeParams p) {
   constexpr uint32_t kIdescQK = make_idesc_bf16(128, kLdKeys, false, false);
   constexpr uint32_t kIdescPV = make_idesc_bf16(128, NH, true, false);
+  constexpr int kScoreCols = NH > 32 ? 2 : 1;               // warps per half page that hold heads
+  constexpr int kTeam = 32 * (kScoreCols + 4);              // scoring and rescaling threads
   constexpr int kQSlab = NH * 128;                          // bytes of one 64-column slab of Q (and of one P buffer)
   extern __shared__ uint8_t ld_raw[];
   uint8_t* sm = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(ld_raw) + 1023) & ~uintptr_t(1023));
@@ -85,10 +92,11 @@ __global__ void __launch_bounds__(kLdThreads) latent_decode_kernel(const __grid_
   uint8_t* ring = sP + 2 * kQSlab;                          // [ring][64 keys][128 B]
   __shared__ uint64_t full_bar[kLdBars], empty_bar[kLdBars], s_bar[2], pv_bar[2], p_bar[2];
   __shared__ uint32_t tmem_slot;
-  __shared__ float s_alpha[2][NH], s_l[NH];
+  __shared__ float s_alpha[2][NH], s_max[2][NH], s_sum[2][NH];
   __shared__ int s_table[kLdTableCap];
 
-  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+  const int tid = threadIdx.x, lane = tid & 31;
+  const int warp = __shfl_sync(0xFFFFFFFFu, tid >> 5, 0);      // known to be uniform: the issue loops run on it
   const int h0 = blockIdx.x * NH, b = blockIdx.y, split = blockIdx.z;
   int n = p.seq_lens[b];
   {
@@ -112,7 +120,7 @@ __global__ void __launch_bounds__(kLdThreads) latent_decode_kernel(const __grid_
   if (tid == 0) {
     tma_prefetch_desc(&p.tma_c);
     for (int i = 0; i < kLdBars; ++i) { mbar_init(&full_bar[i], 1); mbar_init(&empty_bar[i], 1); }
-    for (int i = 0; i < 2; ++i) { mbar_init(&s_bar[i], 1); mbar_init(&pv_bar[i], 1); mbar_init(&p_bar[i], 128); }
+    for (int i = 0; i < 2; ++i) { mbar_init(&s_bar[i], 1); mbar_init(&pv_bar[i], 1); mbar_init(&p_bar[i], kTeam); }
     fence_barrier_init();
   }
   if (warp == 0) {
@@ -135,9 +143,9 @@ __global__ void __launch_bounds__(kLdThreads) latent_decode_kernel(const __grid_
   const uint32_t tmem_base = tmem_slot;
   const uint32_t tO = tmem_base + 128u;                     // S buffers at columns 0 and 64
 
-  if (warp == 5) {
+  if (warp == 7) {
     // ------------------------------------ TMA producer ---------------------------------------
-    if (lane == 0) {
+    if (elect_one()) {
       bool ok = true;
       int slot = 0;                                         // ring slot of the next slab
       int room = p.ring;                                    // free ring slots
@@ -170,191 +178,206 @@ __global__ void __launch_bounds__(kLdThreads) latent_decode_kernel(const __grid_
         }
       }
     }
-  } else if (warp == 4) {
-    // ------------------------------------ MMA issuer -----------------------------------------
-    if (lane == 0 && n_tiles > 0) {
-      // descriptors differ in their address field only: base + byte offset / 16
-      const uint64_t dQ = make_smem_desc(smem_u32(sQ), 16, 1024), dR = make_smem_desc(smem_u32(ring), 16, 1024);
-      const uint64_t dC = make_smem_desc(smem_u32(ring), kLdSlab, 1024), dP = make_smem_desc(smem_u32(sP), 16, 1024);
-      int qk_slot = 0, pv_slot = 0;                         // ring slots of the next page to score / to accumulate
-      auto issue_qk = [&](int j) -> bool {
-        if (!mbar_wait(&full_bar[j % kLdBars], (j / kLdBars) & 1u, p.status)) return false;
-        tc_fence_after_sync();
-        const uint32_t dS = tmem_base + static_cast<uint32_t>((j & 1) * 64);
-        int slot = qk_slot;
-        for (int c = 0; c < p.slabs; ++c) {                 // columns past the row are zero in both operands
-          const uint64_t a = dQ + static_cast<uint64_t>(c * (kQSlab >> 4)), k = dR + static_cast<uint64_t>(slot * (kLdSlab >> 4));
+  } else if (warp == 6 || warp == 8) {
+    // ------------------------------------ MMA issuers ----------------------------------------
+    // descriptors differ in their address field only (the low word): base + byte offset / 16
+    const uint32_t hiK = static_cast<uint32_t>(make_smem_desc(0, 16, 1024) >> 32), loK = static_cast<uint32_t>(make_smem_desc(0, 16, 1024));
+    const uint32_t hiC = static_cast<uint32_t>(make_smem_desc(0, kLdSlab, 1024) >> 32);
+    const uint32_t loC = static_cast<uint32_t>(make_smem_desc(0, kLdSlab, 1024));
+    auto desc = [](uint32_t hi, uint32_t lo) { return (static_cast<uint64_t>(hi) << 32) | lo; };
+    const uint32_t aRing = smem_u32(ring) >> 4;
+    if (warp == 6) {
+      if (elect_one()) {
+        const uint32_t dQ = loK + (smem_u32(sQ) >> 4), dR = loK + aRing;
+        int start = 0;                                      // ring slot of the page
+        for (int j = 0; j < n_tiles; ++j) {
+          // S buffer j & 1 was read for page j - 2: its weights have been reported
+          if (j >= 2 && !mbar_wait(&p_bar[j & 1], ((j - 2) >> 1) & 1u, p.status)) break;
+          if (!mbar_wait(&full_bar[j % kLdBars], (j / kLdBars) & 1u, p.status)) break;
+          tc_fence_after_sync();
+          const uint32_t dS = tmem_base + static_cast<uint32_t>((j & 1) * 64);
+          int slot = start;
+          for (int c = 0; c < p.slabs; ++c) {               // columns past the row are zero in both operands
+            const uint32_t a = dQ + static_cast<uint32_t>(c * (kQSlab >> 4)), k = dR + static_cast<uint32_t>(slot * (kLdSlab >> 4));
 #pragma unroll
-          for (int kk = 0; kk < 4; ++kk) tc_mma_f16_ss(dS, a + kk * 2, k + kk * 2, kIdescQK, (c | kk) != 0 ? 1u : 0u);
-          if (++slot == p.ring) slot = 0;
+            for (int kk = 0; kk < 4; ++kk)
+              tc_mma_f16_ss(dS, desc(hiK, a + kk * 2), desc(hiK, k + kk * 2), kIdescQK, (c | kk) != 0 ? 1u : 0u);
+            if (++slot == p.ring) slot = 0;
+          }
+          start += p.slots;
+          if (start >= p.ring) start -= p.ring;
+          tc_commit(&s_bar[j & 1]);
         }
-        qk_slot += p.slots;
-        if (qk_slot >= p.ring) qk_slot -= p.ring;
-        tc_commit(&s_bar[j & 1]);
-        return true;
-      };
-      bool ok = issue_qk(0);
-      for (int j = 0; j < n_tiles && ok; ++j) {
-        bool ahead = j + 1 >= n_tiles;
-        if (!ahead && mbar_test_wait(&full_bar[(j + 1) % kLdBars], ((j + 1) / kLdBars) & 1u)) {
-          ok = issue_qk(j + 1);                             // the next page is here: score it under this page's softmax
-          ahead = true;
-          if (!ok) break;
-        }
-        // (one barrier per P buffer: the softmax warps may finish page j + 1 before this thread looks at page j)
-        ok = mbar_wait(&p_bar[j & 1], (j >> 1) & 1u, p.status);
-        if (!ok) break;
+      }
+    } else if (elect_one()) {
+      const uint32_t dC = loC + aRing, dP = loK + (smem_u32(sP) >> 4);
+      int start = 0;
+      for (int j = 0; j < n_tiles; ++j) {
+        // one barrier per P buffer: the softmax warps may finish page j + 1 before this thread looks at page j
+        if (!mbar_wait(&p_bar[j & 1], (j >> 1) & 1u, p.status)) break;
         tc_fence_after_sync();
-        const uint64_t bP = dP + static_cast<uint64_t>((j & 1) * (kQSlab >> 4));
-        int slot = pv_slot;
+        const uint32_t bP = dP + static_cast<uint32_t>((j & 1) * (kQSlab >> 4));
+        int slot = start;
         for (int m = 0; m < p.chunks; ++m) {
-          const uint64_t aC = dC + static_cast<uint64_t>(slot * (kLdSlab >> 4));
+          const uint32_t aC = dC + static_cast<uint32_t>(slot * (kLdSlab >> 4));
 #pragma unroll
           for (int kk = 0; kk < kLdKeys / 16; ++kk)
-            tc_mma_f16_ss(tO + static_cast<uint32_t>(m * NH), aC + kk * (2048 >> 4), bP + kk * 2, kIdescPV,
-                          (j | kk) != 0 ? 1u : 0u);
+            tc_mma_f16_ss(tO + static_cast<uint32_t>(m * NH), desc(hiC, aC + kk * (2048 >> 4)), desc(hiK, bP + kk * 2),
+                          kIdescPV, (j | kk) != 0 ? 1u : 0u);
           slot += 2;
           if (slot >= p.ring) slot -= p.ring;
         }
-        pv_slot += p.slots;
-        if (pv_slot >= p.ring) pv_slot -= p.ring;
+        start += p.slots;
+        if (start >= p.ring) start -= p.ring;
         tc_commit(&pv_bar[j & 1]);
         tc_commit(&empty_bar[j % kLdBars]);
-        if (!ahead) ok = issue_qk(j + 1);
       }
     }
-  } else {
-    // ------------------------------------ softmax --------------------------------------------
-    const uint32_t lane_off = static_cast<uint32_t>(warp * 32) << 16;
-    const bool scoring = warp * 32 < NH;                    // warp-uniform: this warp's lanes hold heads
+    __syncwarp();
+  } else if ((warp & 3) < kScoreCols || warp < 4) {
+    // ------------------------------------ softmax, rescaling, output -------------------------
+    const uint32_t lane_off = static_cast<uint32_t>((warp & 3) * 32) << 16;
+    const bool scoring = (warp & 3) < kScoreCols;           // warp-uniform: the lanes of this warp hold heads
+    const int half = warp >> 2;                             // keys half * 32 .. + 31 of every page
+    const int hr = (warp & 3) * 32 + lane;                  // head row = TMEM lane of S
+    const bool head = scoring && hr < NH;
     float m_used = -1.0e29f, l_sum = 0.f;
     bool ok = true;
     for (int j = 0; j < n_tiles; ++j) {
-      const int page = table[j];
-      const bool page_ok = page >= 0 && page < p.num_blocks;
-      const int k0 = (pg0 + j) * kLdKeys;
-      // P buffer j & 1 was read by the product of page j - 2
-      if (j >= 2) {
-        ok = ok && mbar_wait(&pv_bar[j & 1], ((j - 2) >> 1) & 1u, p.status);
-        ok = __all_sync(0xFFFFFFFFu, ok);
-      }
-      float alpha = 1.f;
-      bool rescale = false;
+      uint32_t s[32];
+      float mx = -1.0e30f;
       if (scoring) {
         ok = ok && mbar_wait(&s_bar[j & 1], (j >> 1) & 1u, p.status);
         ok = __all_sync(0xFFFFFFFFu, ok);
         if (ok) {
           tc_fence_after_sync();
-          uint32_t s[64];
-          {
-            uint32_t(&c0)[32] = *reinterpret_cast<uint32_t(*)[32]>(&s[0]);
-            uint32_t(&c1)[32] = *reinterpret_cast<uint32_t(*)[32]>(&s[32]);
-            const uint32_t tS = tmem_base + lane_off + static_cast<uint32_t>((j & 1) * 64);
-            tmem_ld32(tS, c0);
-            tmem_ld32(tS + 32, c1);
-            tc_wait_ld();
-          }
-          float mx = -1.0e30f;
-          if (k0 < first || k0 + kLdKeys > n || !page_ok) {
+          tmem_ld32(tmem_base + lane_off + static_cast<uint32_t>((j & 1) * 64 + half * 32), s);
+          tc_wait_ld();
+          const int page = table[j];
+          const bool page_ok = page >= 0 && page < p.num_blocks;
+          const int k0 = (pg0 + j) * kLdKeys + half * 32;
+          if (k0 < first || k0 + 32 > n || !page_ok) {
 #pragma unroll
-            for (int i = 0; i < 64; ++i)
+            for (int i = 0; i < 32; ++i)
               if (k0 + i < first || k0 + i >= n || !page_ok) s[i] = 0xFF800000u;
           }
+          float t[16];
 #pragma unroll
-          for (int i = 0; i < 64; ++i) mx = fmaxf(mx, __uint_as_float(s[i]));
+          for (int i = 0; i < 16; ++i) t[i] = fmaxf(__uint_as_float(s[2 * i]), __uint_as_float(s[2 * i + 1]));
+#pragma unroll
+          for (int w = 8; w > 0; w >>= 1)
+#pragma unroll
+            for (int i = 0; i < w; ++i) t[i] = fmaxf(t[i], t[i + w]);
+          mx = fmaxf(t[0], -1.0e30f);
           mx = mx > -0.5e30f ? mx * p.scale_log2 : -1.0e30f;
-          if (mx > m_used + 8.f) {                          // lazy: the reference maximum moves in large steps only
-            alpha = ld_exp2(m_used - mx);
-            m_used = mx;
-            rescale = j > 0;
-          }
-          uint32_t pk[32];
-          float ls = 0.f;
-#pragma unroll
-          for (int i = 0; i < 32; ++i) {
-            const float e0 = ld_exp2(fmaf(__uint_as_float(s[2 * i]), p.scale_log2, -m_used));
-            const float e1 = ld_exp2(fmaf(__uint_as_float(s[2 * i + 1]), p.scale_log2, -m_used));
-            const uint32_t bits = pack_bf16(e0, e1);
-            pk[i] = bits;
-            ls += __uint_as_float(bits << 16) + __uint_as_float(bits & 0xFFFF0000u);   // the weights as multiplied
-          }
-          l_sum = l_sum * alpha + ls;
-          const int r = tid;                                // head row
-          if (r < NH) {
-            s_alpha[j & 1][r] = alpha;
-            uint8_t* row = sP + (j & 1) * kQSlab + r * 128;
-#pragma unroll
-            for (int c = 0; c < 8; ++c)
-              *reinterpret_cast<uint4*>(row + ((c ^ (r & 7)) << 4)) =
-                  make_uint4(pk[4 * c], pk[4 * c + 1], pk[4 * c + 2], pk[4 * c + 3]);
-          } else {
-            rescale = false;                                // lanes past NH hold no head
-          }
-          __syncwarp();
           tc_fence_before_sync();
         }
       }
-      if (ld_barrier_or(rescale || !ok)) {
-        ok = !ld_barrier_or(!ok);                           // all 128 threads agree
+      if (ld_barrier_or<kTeam>((head && mx > m_used + 8.f) || !ok)) {
+        ok = !ld_barrier_or<kTeam>(!ok);                    // everyone agrees
         if (!ok) break;
+        if (head) s_max[half][hr] = mx;
         // O^T holds sums relative to the old maxima: the previous product must be complete before it is scaled
-        ok = mbar_wait(&pv_bar[(j - 1) & 1], ((j - 1) >> 1) & 1u, p.status);
-        ok = __all_sync(0xFFFFFFFFu, ok);
-        ok = !ld_barrier_or(!ok);
-        if (!ok) break;
-        tc_fence_after_sync();
-        for (int m = 0; m < p.chunks; ++m) {
-#pragma unroll
-          for (int g = 0; g < NH; g += 16) {
-            uint32_t o[16];
-            tmem_ld16(tO + lane_off + static_cast<uint32_t>(m * NH + g), o);
-            tc_wait_ld();
-#pragma unroll
-            for (int i = 0; i < 16; ++i) o[i] = __float_as_uint(__uint_as_float(o[i]) * s_alpha[j & 1][g + i]);
-            tmem_st16(tO + lane_off + static_cast<uint32_t>(m * NH + g), o);
-          }
+        if (j > 0) {
+          ok = mbar_wait(&pv_bar[(j - 1) & 1], ((j - 1) >> 1) & 1u, p.status);
+          ok = __all_sync(0xFFFFFFFFu, ok);
         }
-        tc_wait_st();
-        tc_fence_before_sync();
+        ok = !ld_barrier_or<kTeam>(!ok);
+        if (!ok) break;
+        if (head) {
+          const float all = fmaxf(s_max[0][hr], s_max[1][hr]);
+          float alpha = 1.f;
+          if (all > m_used + 8.f) {
+            alpha = ld_exp2(m_used - all);
+            m_used = all;
+            l_sum *= alpha;
+          }
+          if (half == 0) s_alpha[j & 1][hr] = alpha;
+        }
+        ld_barrier_or<kTeam>(false);
+        if (warp < 4 && j > 0) {
+          tc_fence_after_sync();
+          for (int m = 0; m < p.chunks; ++m) {
+#pragma unroll
+            for (int g = 0; g < NH; g += 16) {
+              uint32_t o[16];
+              __syncwarp();
+              tmem_ld16(tO + lane_off + static_cast<uint32_t>(m * NH + g), o);
+              tc_wait_ld();
+#pragma unroll
+              for (int i = 0; i < 16; ++i) o[i] = __float_as_uint(__uint_as_float(o[i]) * s_alpha[j & 1][g + i]);
+              tmem_st16(tO + lane_off + static_cast<uint32_t>(m * NH + g), o);
+            }
+          }
+          tc_wait_st();
+          tc_fence_before_sync();
+        }
       }
-      fence_proxy_async_smem();
-      mbar_arrive(&p_bar[j & 1]);
+      if (scoring) {
+        // P buffer j & 1 was read by the product of page j - 2
+        if (j >= 2) {
+          ok = mbar_wait(&pv_bar[j & 1], ((j - 2) >> 1) & 1u, p.status);
+          ok = __all_sync(0xFFFFFFFFu, ok);                 // a failure is agreed on at the next barrier
+        }
+        uint32_t pk[16];
+        float ls[4] = {0.f, 0.f, 0.f, 0.f};
+#pragma unroll
+        for (int i = 0; i < 16; ++i) {
+          const float e0 = ld_exp2(fmaf(__uint_as_float(s[2 * i]), p.scale_log2, -m_used));
+          const float e1 = ld_exp2(fmaf(__uint_as_float(s[2 * i + 1]), p.scale_log2, -m_used));
+          pk[i] = pack_bf16(e0, e1);
+          ls[i & 3] += __uint_as_float(pk[i] << 16) + __uint_as_float(pk[i] & 0xFFFF0000u);   // the weights as multiplied
+        }
+        l_sum += (ls[0] + ls[1]) + (ls[2] + ls[3]);
+        if (head && ok) {
+          uint8_t* row = sP + (j & 1) * kQSlab + hr * 128;
+#pragma unroll
+          for (int c = 0; c < 4; ++c)
+            *reinterpret_cast<uint4*>(row + (((4 * half + c) ^ (hr & 7)) << 4)) =
+                make_uint4(pk[4 * c], pk[4 * c + 1], pk[4 * c + 2], pk[4 * c + 3]);
+        }
+        __syncwarp();
+        fence_proxy_async_smem();
+      }
+      if (ok) mbar_arrive(&p_bar[j & 1]);
     }
     if (ok && n_tiles > 0) ok = mbar_wait(&pv_bar[(n_tiles - 1) & 1], ((n_tiles - 1) >> 1) & 1u, p.status);
     ok = __all_sync(0xFFFFFFFFu, ok);
-    if (tid < NH) s_l[tid] = l_sum;
-    ok = !ld_barrier_or(!ok);
+    if (head) s_sum[half][hr] = l_sum;
+    ok = !ld_barrier_or<kTeam>(!ok);
     // after a wait that ran out (status set) the outputs are still written, as zeros
-    if (tid < NH && h0 + tid < p.heads && p.splits > 1) {
-      const int64_t base = (static_cast<int64_t>(b) * p.heads + h0 + tid) * p.splits + split;
+    if (head && half == 0 && h0 + hr < p.heads && p.splits > 1) {
+      const int64_t base = (static_cast<int64_t>(b) * p.heads + h0 + hr) * p.splits + split;
       p.partial_ml[base * 2] = ok ? m_used : -1.0e29f;
-      p.partial_ml[base * 2 + 1] = ok ? l_sum : 0.f;
+      p.partial_ml[base * 2 + 1] = ok ? s_sum[0][hr] + s_sum[1][hr] : 0.f;
     }
-    tc_fence_after_sync();
-    for (int m = 0; m < p.chunks; ++m) {
-      const int dim = m * 128 + tid;
+    if (warp < 4) {
+      tc_fence_after_sync();
+      for (int m = 0; m < p.chunks; ++m) {
+        const int dim = m * 128 + tid;
 #pragma unroll
-      for (int g = 0; g < NH; g += 16) {
-        uint32_t o[16];
-        __syncwarp();
-        if (ok && n_tiles > 0) {
-          tmem_ld16(tO + lane_off + static_cast<uint32_t>(m * NH + g), o);
-          tc_wait_ld();
-        } else {
+        for (int g = 0; g < NH; g += 16) {
+          uint32_t o[16];
+          __syncwarp();
+          if (ok && n_tiles > 0) {
+            tmem_ld16(tO + lane_off + static_cast<uint32_t>(m * NH + g), o);
+            tc_wait_ld();
+          } else {
 #pragma unroll
-          for (int i = 0; i < 16; ++i) o[i] = 0u;
-        }
-        if (dim < p.kv_rank) {
+            for (int i = 0; i < 16; ++i) o[i] = 0u;
+          }
+          if (dim < p.kv_rank) {
 #pragma unroll
-          for (int i = 0; i < 16; ++i) {
-            const int h = h0 + g + i;
-            if (h < p.heads) {
-              const float v = __uint_as_float(o[i]);
-              if (p.splits > 1) {
-                p.partial_o[((static_cast<int64_t>(b) * p.heads + h) * p.splits + split) * p.kv_rank + dim] = v;
-              } else {
-                const float l = s_l[g + i];
-                p.out[(static_cast<int64_t>(h) * p.rows_pad + b) * p.kv_rank + dim] = __float2bfloat16(l > 0.f ? v / l : 0.f);
+            for (int i = 0; i < 16; ++i) {
+              const int h = h0 + g + i;
+              if (h < p.heads) {
+                const float v = __uint_as_float(o[i]);
+                if (p.splits > 1) {
+                  p.partial_o[((static_cast<int64_t>(b) * p.heads + h) * p.splits + split) * p.kv_rank + dim] = v;
+                } else {
+                  const float l = s_sum[0][g + i] + s_sum[1][g + i];
+                  p.out[(static_cast<int64_t>(h) * p.rows_pad + b) * p.kv_rank + dim] = __float2bfloat16(l > 0.f ? v / l : 0.f);
+                }
               }
             }
           }
