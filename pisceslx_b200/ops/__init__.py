@@ -15,6 +15,7 @@ from typing import Dict, Optional
 import torch
 
 _SO = Path(__file__).resolve().parent / "_yv_ops.so"
+_LAYERED_SO = _SO.with_name("_yv_layered.so")
 _lock = threading.Lock()
 _loaded = False
 _status: Dict[int, torch.Tensor] = {}
@@ -38,22 +39,24 @@ def extension_built() -> bool:
     return _SO.exists()
 
 
-def load_extension(build_if_missing: bool = False) -> None:
-    """Load ``_yv_ops.so`` (idempotent).  Raises ``RuntimeError`` when it has not been built."""
+def load_extension(build_if_missing: bool = False, layered: bool = False) -> None:
+    """Load ``_yv_ops.so`` (idempotent).  Raises ``RuntimeError`` when it has not been built.  With ``layered`` a
+    process that runs nothing but layered models takes the smaller ``_yv_layered.so`` when the full one is missing."""
     global _loaded
     if _loaded:
         return
     with _lock:
         if _loaded:
             return
-        if not _SO.exists():
+        so = _LAYERED_SO if layered and not _SO.exists() else _SO
+        if not so.exists():
             if build_if_missing or os.environ.get("YV_BUILD_ON_IMPORT") == "1":
                 from .build import build
-                build()
+                build(layered=so == _LAYERED_SO)
             else:
                 raise RuntimeError(
-                    f"{_SO} is missing: run `python -m pisceslx_b200.ops.build` (or __graft_entry__.build()) first")
-        torch.ops.load_library(str(_SO))
+                    f"{so} is missing: run `python -m pisceslx_b200.ops.build` (or __graft_entry__.build()) first")
+        torch.ops.load_library(str(so))
         _loaded = True
 
 

@@ -18,10 +18,14 @@ HERE = Path(__file__).resolve().parent
 CSRC = HERE / "csrc"
 OBJ = HERE / "build"
 SO = HERE / "_yv_ops.so"
+LAYERED_SO = HERE / "_yv_layered.so"
 
 CUDA_SOURCES = ["gemm.cu", "elementwise.cu", "moe.cu", "loss_optim.cu", "attention.cu", "comm.cu", "noalloc.cu", "ssm.cu", "pq_film.cu",
                 "stream.cu", "latent.cu"]
 CPP_SOURCES = ["binding.cpp"]
+# the subset that serves layered models (same operators, a library of its own)
+LAYERED_CUDA_SOURCES = ["gemm.cu", "elementwise.cu", "stream.cu", "latent.cu"]
+LAYERED_CPP_SOURCES = ["binding_layered.cpp"]
 NVCC_FLAGS = ["-gencode", "arch=compute_100a,code=sm_100a", "-lineinfo", "-O3", "-std=c++17",
               "--expt-relaxed-constexpr", "-Xcompiler", "-fPIC", "-diag-suppress", "550"]
 
@@ -66,7 +70,8 @@ def _run(cmd: List[str]) -> None:
         raise RuntimeError(f"build step failed: {cmd[0]} {cmd[-1]}")
 
 
-def build(verbose: bool = False, force: bool = False) -> Path:
+def build(verbose: bool = False, force: bool = False, layered: bool = False) -> Path:
+    """Compile what has changed and link ``_yv_ops.so`` (``layered``: the subset ``_yv_layered.so``)."""
     import torch
     from torch.utils import cpp_extension as ce
 
@@ -75,7 +80,8 @@ def build(verbose: bool = False, force: bool = False) -> Path:
     nvcc = os.path.join(_cuda_home(), "bin", "nvcc")
     jobs = []
     objs: List[Path] = []
-    for name in CUDA_SOURCES:
+    so = LAYERED_SO if layered else SO
+    for name in LAYERED_CUDA_SOURCES if layered else CUDA_SOURCES:
         src = CSRC / name
         if not src.exists():
             continue
@@ -87,7 +93,7 @@ def build(verbose: bool = False, force: bool = False) -> Path:
     for p in ce.include_paths("cuda"):
         inc += ["-isystem", p]
     cxx = _host_cxx()
-    for name in CPP_SOURCES:
+    for name in LAYERED_CPP_SOURCES if layered else CPP_SOURCES:
         src = CSRC / name
         obj = OBJ / (name + ".o")
         objs.append(obj)
@@ -101,14 +107,14 @@ def build(verbose: bool = False, force: bool = False) -> Path:
             print(" ".join(j))
     with ThreadPoolExecutor(max_workers=min(8, max(1, len(jobs)))) as ex:
         list(ex.map(_run, jobs))
-    if jobs or not SO.exists() or force:
+    if jobs or not so.exists() or force:
         torch_lib = os.path.join(os.path.dirname(torch.__file__), "lib")
-        cmd = [cxx, "-shared", "-o", str(SO)] + [str(o) for o in objs] + [
+        cmd = [cxx, "-shared", "-o", str(so)] + [str(o) for o in objs] + [
             f"-L{torch_lib}", "-ltorch", "-ltorch_cpu", "-ltorch_cuda", "-lc10", "-lc10_cuda",
             f"-L{os.path.join(_cuda_home(), 'lib64')}", "-lcudart", "-lstdc++", f"-Wl,-rpath,{torch_lib}"]
         _run(cmd)
-        _check_dynamic_libstdcxx(SO)
-    return SO
+        _check_dynamic_libstdcxx(so)
+    return so
 
 
 if __name__ == "__main__":

@@ -1,74 +1,9 @@
 // PyTorch bindings (torch.ops.yv.*) for the sm_100a kernels.  Every op checks device, dtype, layout
 // and alignment on the host, passes raw pointers plus the current stream to a launcher, and raises on
 // a non-zero launcher code.  No op allocates: outputs and scratch are passed in by the Python layer.
-#include <ATen/cuda/CUDAContext.h>
-#include <c10/cuda/CUDAGuard.h>
-#include <torch/library.h>
-#include <torch/torch.h>
-
-#include "yv_ops.h"
+#include "binding_gemm.inc"
 
 namespace {
-
-using torch::Tensor;
-
-inline cudaStream_t cur_stream() { return at::cuda::getCurrentCUDAStream().stream(); }
-
-inline void check_cuda(const Tensor& t, const char* name) {
-  TORCH_CHECK(t.is_cuda(), name, " must be a CUDA tensor");
-}
-inline void check_bf16(const Tensor& t, const char* name) {
-  check_cuda(t, name);
-  TORCH_CHECK(t.scalar_type() == at::kBFloat16, name, " must be bfloat16");
-}
-inline void check_f32(const Tensor& t, const char* name) {
-  check_cuda(t, name);
-  TORCH_CHECK(t.scalar_type() == at::kFloat, name, " must be float32");
-}
-inline void check_i32(const Tensor& t, const char* name) {
-  check_cuda(t, name);
-  TORCH_CHECK(t.scalar_type() == at::kInt, name, " must be int32");
-}
-inline void check_rc(int rc, const char* what) {
-  TORCH_CHECK(rc == 0, "pisceslx_b200 kernel launch failed: ", what, " rc=", rc,
-              rc > 0 ? std::string(" (") + cudaGetErrorString(static_cast<cudaError_t>(rc)) + ")" : std::string());
-}
-inline const void* optp(const c10::optional<Tensor>& t) { return t.has_value() ? t->data_ptr() : nullptr; }
-inline uint32_t* statusp(const c10::optional<Tensor>& t) {
-  return t.has_value() ? reinterpret_cast<uint32_t*>(t->data_ptr()) : nullptr;
-}
-inline int dt_code(const Tensor& t) {
-  if (t.scalar_type() == at::kFloat) return 1;
-  TORCH_CHECK(t.scalar_type() == at::kBFloat16, "expected bf16 or fp32 tensor");
-  return 0;
-}
-
-// ------------------------------------------------------------------------------------------------
-// GEMM.  a: [M,K] (a_mn=false) or [K,M] (a_mn=true); b: [N,K] (b_mn=false) or [K,N] (b_mn=true); 2-D, inner
-// stride 1.  c: [M,N] bf16 or fp32.
-// ------------------------------------------------------------------------------------------------
-void gemm(const Tensor& a, const Tensor& b, Tensor c, bool a_mn, bool b_mn, bool accumulate, int64_t bn,
-          const c10::optional<Tensor>& status) {
-  check_bf16(a, "a"); check_bf16(b, "b"); check_cuda(c, "c");
-  TORCH_CHECK(a.dim() == 2 && b.dim() == 2 && c.dim() == 2, "gemm operands must be 2-D");
-  TORCH_CHECK(a.stride(1) == 1 && b.stride(1) == 1 && c.stride(1) == 1, "gemm operands need unit inner stride");
-  const c10::cuda::CUDAGuard guard(a.device());
-  yv::GemmArgs g;
-  g.a = a.data_ptr(); g.b = b.data_ptr(); g.c = c.data_ptr();
-  g.a_mn = a_mn; g.b_mn = b_mn;
-  g.M = static_cast<int>(a_mn ? a.size(1) : a.size(0));
-  g.K = static_cast<int>(a_mn ? a.size(0) : a.size(1));
-  g.N = static_cast<int>(b_mn ? b.size(1) : b.size(0));
-  const int64_t kb = b_mn ? b.size(0) : b.size(1);
-  TORCH_CHECK(kb == g.K, "gemm: inner dimensions differ: ", g.K, " vs ", kb);
-  TORCH_CHECK(c.size(0) == g.M && c.size(1) == g.N, "gemm: output shape mismatch");
-  g.lda = a.stride(0); g.ldb = b.stride(0); g.ldc = c.stride(0);
-  g.out_fp32 = dt_code(c);
-  g.accumulate = accumulate ? 1 : 0;
-  g.bn = static_cast<int>(bn);
-  g.status = statusp(status);
-  check_rc(yv::launch_gemm(g, cur_stream()), "gemm");
-}
 
 // Grouped along M: a [rows_total, K] expert-sorted/padded; b [E, N, K] (b_mn=false) or [E, K, N] (b_mn=true);
 // c [rows_total, N].
@@ -126,37 +61,6 @@ void gemm_grouped_k(const Tensor& a, const Tensor& b, Tensor c, const Tensor& se
   g.status = statusp(status);
   check_rc(yv::launch_gemm(g, cur_stream()), "gemm_grouped_k");
 }
-
-// Batched: a [G, M, K] (or [G, K, M] when a_mn), b [G, N, K] (or [G, K, N] when b_mn), c [G, M, N]; contiguous.
-void gemm_batched(const Tensor& a, const Tensor& b, Tensor c, bool a_mn, bool b_mn, bool accumulate, int64_t bn,
-                  const c10::optional<Tensor>& status, bool symmetric) {
-  check_bf16(a, "a"); check_bf16(b, "b"); check_cuda(c, "c");
-  // groups are stacked along the rows: a row pitch is allowed, a gap between groups is not
-  auto stacked = [](const Tensor& t) {
-    return t.dim() == 3 && t.stride(2) == 1 && (t.size(0) == 1 || t.stride(0) == t.size(1) * t.stride(1));
-  };
-  TORCH_CHECK(stacked(a) && stacked(b) && stacked(c), "gemm_batched: stacked 3-D operands expected");
-  TORCH_CHECK(a.size(0) == b.size(0) && a.size(0) == c.size(0), "gemm_batched: batch sizes differ");
-  const c10::cuda::CUDAGuard guard(a.device());
-  yv::GemmArgs g;
-  g.a = a.data_ptr(); g.b = b.data_ptr(); g.c = c.data_ptr();
-  g.a_mn = a_mn; g.b_mn = b_mn;
-  g.mode = 3;
-  g.num_groups = static_cast<int>(a.size(0));
-  g.M = static_cast<int>(a_mn ? a.size(2) : a.size(1));
-  g.K = static_cast<int>(a_mn ? a.size(1) : a.size(2));
-  g.N = static_cast<int>(b_mn ? b.size(2) : b.size(1));
-  TORCH_CHECK((b_mn ? b.size(1) : b.size(2)) == g.K, "gemm_batched: K mismatch");
-  TORCH_CHECK(c.size(1) == g.M && c.size(2) == g.N, "gemm_batched: output shape mismatch");
-  g.lda = a.stride(1); g.ldb = b.stride(1); g.ldc = c.stride(1);
-  g.out_fp32 = dt_code(c);
-  g.accumulate = accumulate ? 1 : 0;
-  g.bn = static_cast<int>(bn);
-  g.status = statusp(status);
-  g.symmetric = symmetric;
-  check_rc(yv::launch_gemm(g, cur_stream()), "gemm_batched");
-}
-
 // c[g] = ec * (a[g] @ b[g]^T) + eb * cin[g] + ea * I   (square [n, n] outputs, n a multiple of 128): the
 // Newton-Schulz polynomial b A + c A^2 + a I formed in the epilogue of the A A product
 void gemm_batched_affine(const Tensor& a, const Tensor& b, const Tensor& cin, Tensor c, double ea, double eb, double ec,
@@ -293,34 +197,6 @@ void add(const Tensor& a, const Tensor& b, Tensor out) {
   check_bf16(a, "a"); check_bf16(b, "b"); check_bf16(out, "out");
   const c10::cuda::CUDAGuard guard(a.device());
   check_rc(yv::launch_add(a.data_ptr(), b.data_ptr(), out.data_ptr(), a.numel(), cur_stream()), "add");
-}
-
-// Split-K product for skinny activations: y[M,N] = a[M,K] @ b[N,K]^T (+ bias) with the K range cut into
-// seg_offsets.numel()-1 slices (offsets are multiples of 64), each reduced by its own CTAs into the fp32 workspace
-// ws [slices, ceil128(M), N]; a second kernel sums the slices in a fixed order (bit-reproducible).
-void gemm_splitk(const Tensor& a, const Tensor& b, Tensor ws, const Tensor& seg_offsets,
-                 const c10::optional<Tensor>& bias, Tensor out, const c10::optional<Tensor>& status) {
-  check_bf16(a, "a"); check_bf16(b, "b"); check_f32(ws, "ws"); check_i32(seg_offsets, "seg_offsets"); check_bf16(out, "out");
-  TORCH_CHECK(a.dim() == 2 && b.dim() == 2 && a.stride(1) == 1 && b.stride(1) == 1 && out.is_contiguous() &&
-              ws.is_contiguous(), "gemm_splitk: a [M,K], b [N,K] with unit inner stride, contiguous ws and out");
-  const int slices = static_cast<int>(seg_offsets.numel()) - 1;
-  const int M = static_cast<int>(a.size(0)), K = static_cast<int>(a.size(1)), N = static_cast<int>(b.size(0));
-  const int m_pad = (M + 127) / 128 * 128;
-  TORCH_CHECK(slices >= 1 && b.size(1) == K && out.size(0) == M && out.size(1) == N, "gemm_splitk: shape mismatch");
-  TORCH_CHECK(ws.numel() >= static_cast<int64_t>(slices) * m_pad * N, "gemm_splitk: workspace too small");
-  const c10::cuda::CUDAGuard guard(a.device());
-  yv::GemmArgs g;
-  g.a = a.data_ptr(); g.b = b.data_ptr(); g.c = ws.data_ptr();
-  g.M = M; g.N = N; g.K = K;
-  g.lda = a.stride(0); g.ldb = b.stride(0); g.ldc = N;
-  g.out_fp32 = 1;
-  g.mode = 4;
-  g.num_groups = slices;
-  g.seg_offsets = seg_offsets.data_ptr<int>();
-  g.status = statusp(status);
-  check_rc(yv::launch_gemm(g, cur_stream()), "gemm_splitk");
-  check_rc(yv::launch_splitk_reduce(ws.data_ptr<float>(), bias.has_value() ? bias->data_ptr() : nullptr,
-                                    out.data_ptr(), slices, M, m_pad, N, cur_stream()), "splitk_reduce");
 }
 
 inline void check_fp8(const Tensor& t, const char* name) {

@@ -79,7 +79,7 @@ def main(argv: Optional[List[str]] = None) -> int:
         return 2
     from ..engine.loader import load_model_for_inference
     from ..ops import load_extension
-    load_extension(build_if_missing=True)
+    load_extension(build_if_missing=True, layered=True)
     dtype = DTYPES[args.dtype]
     if dtype == torch.float32:
         torch.backends.cuda.matmul.allow_tf32 = torch.backends.cudnn.allow_tf32 = False
