@@ -103,7 +103,10 @@ class YvRotaryEmbedding(nn.Module):
 
     def tables(self, needed: int, device: torch.device) -> Tuple[torch.Tensor, torch.Tensor]:
         if needed > self.max_position or self.cos.device != device:
-            self._build(max(needed, self.max_position), device)
+            size = max(needed, self.max_position)
+            if needed > self.max_position and self.scaling_type != "dynamic_ntk":
+                size = max(size, 2 * self.max_position)      # sequences grow token by token: not a table per step
+            self._build(size, device)
         return self.cos, self.sin
 
     def forward(self, x: torch.Tensor, positions: torch.Tensor) -> torch.Tensor:

@@ -52,7 +52,7 @@ def _kernel_shares(fn, top: int = 12) -> List[Tuple[str, float, int]]:
     with profile(activities=[ProfilerActivity.CUDA]) as prof:
         fn()
         torch.cuda.synchronize()
-    rows = [(e.key.split("(")[0].replace("void ", "")[:90], e.self_device_time_total, e.count) for e in prof.key_averages()
+    rows = [(e.key.replace("(anonymous namespace)::", "").split("(")[0].replace("void ", "")[:90], e.self_device_time_total, e.count) for e in prof.key_averages()
             if e.self_device_time_total > 0]
     return sorted(rows, key=lambda r: -r[1])[:top]
 
