@@ -18,7 +18,7 @@ import math
 from dataclasses import dataclass, field
 from enum import Enum
 from pathlib import Path
-from typing import Any, Dict, List, Optional
+from typing import Any, Dict, List, Optional, Tuple
 
 import yaml
 
@@ -223,6 +223,11 @@ class YvConfig:
     # ---- layered architectures (``architectures`` fills these from a checkpoint's config.json) ----------------------
     layer_specs: List[Dict[str, Any]] = field(default_factory=list)   # one {"mixer": ..., "mlp": ...} per layer
     token_side_dim: int = 0                 # width of the per-layer token input (0 = none)
+    layer_block: str = "sandwich"           # how a layer joins its branches to the stream (``models.layered.BLOCKS``)
+    layer_loop: Optional[Dict[str, int]] = None   # layers start .. stop - 1 run ``times`` times in a row
+    norm_offset: float = 0.0                # constant added to stored norm weights
+    embedding_norm: bool = True             # the stream starts with the normed embedding ...
+    embedding_scale: float = 1.0            # ... or, without the norm, with the embedding times this
     # ---- task heads ---------------------------------------------------------------------------------------------
     task_classes: int = 256
     classifier_dropout: float = 0.1
@@ -317,20 +322,39 @@ class YvConfig:
         return {"total": int(total), "active": int(active), "embedding": int(emb),
                 "per_layer": int(per_layer_moe if n_moe else per_layer_dense)}
 
+    def layer_runs(self) -> List[Tuple[int, Optional[int], bool]]:
+        """The order in which a layered model's layers run: (layer, number of the pass or None outside the loop, first
+        layer of a pass).  Every run has a cache of its own."""
+        plain = lambda lo, hi: [(i, None, False) for i in range(lo, hi)]
+        if not self.layer_loop:
+            return plain(0, self.n_layer)
+        lo, hi = self.layer_loop["start"], self.layer_loop["stop"]
+        body = [(i, t, i == lo) for t in range(self.layer_loop["times"]) for i in range(lo, hi)]
+        return plain(0, lo) + body + plain(hi, self.n_layer)
+
+    def _count_mixer(self, m: Dict[str, Any]) -> int:
+        H, heads = self.hidden_size, m["heads"]
+        if m["kind"] == "grouped_attention":
+            qkv = heads * m["dim"] + m["kv_heads"] * (m["dim"] + m["vdim"])
+            gate = {"element": heads * m["vdim"], "head": heads}.get(m.get("output_gate"), 0)
+            return (qkv + gate) * H + (qkv if m.get("bias") else 0) + (heads if m.get("sink") else 0) + H * heads * m["vdim"]
+        hd = heads * (m["dim"] + m["rot_dim"])
+        return (H * (m["q_rank"] + m["kv_rank"] + m["rot_dim"] + (heads if m.get("output_gate") else 0)) + hd * m["q_rank"]
+                + heads * (m["dim"] + m["vdim"]) * m["kv_rank"] + H * heads * m["vdim"] + m["q_rank"] + m["kv_rank"])
+
     def _count_layered(self) -> Dict[str, int]:
         H, S = self.hidden_size, self.token_side_dim
+        norms = 2 * H if self.layer_block == "sandwich" else H
         total = 0
         for spec in self.layer_specs:
-            m, f = spec["mixer"], spec["mlp"]
-            hd = m["heads"] * (m["dim"] + m["rot_dim"])
-            total += (H * (m["q_rank"] + m["kv_rank"] + m["rot_dim"] + (m["heads"] if m.get("output_gate") else 0))
-                      + hd * m["q_rank"] + m["heads"] * (m["dim"] + m["vdim"]) * m["kv_rank"] + H * m["heads"] * m["vdim"]
-                      + m["q_rank"] + m["kv_rank"] + 2 * H)
-            total += (2 * H * f["ff"] + 2 * H) if f else 0
+            f = spec["mlp"]
+            total += self._count_mixer(spec["mixer"]) + norms
+            total += ((3 if f["kind"] == "dense_swiglu" else 2) * H * f["ff"] + norms) if f else 0
             total += (2 * H * S + H) if S else 0
         emb = 2 * self.vocab_size * H
         side = self.vocab_size * self.n_layer * S
-        return {"total": int(total + emb + side + 2 * H), "active": int(total + self.vocab_size * H),
+        rest = H * (1 + int(self.embedding_norm)) + (self.layer_loop["times"] * H if self.layer_loop else 0)
+        return {"total": int(total + emb + side + rest), "active": int(total + self.vocab_size * H),
                 "embedding": int(emb + side), "per_layer": int(total // max(self.n_layer, 1))}
 
     def estimate_memory_usage(self, batch: int = 1, seq: int = 4096, bytes_per_param: int = 2,

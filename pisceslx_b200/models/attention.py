@@ -54,9 +54,17 @@ class AttnContext:
     starts: Optional[List[int]] = None
     lens: Optional[List[int]] = None
     slots_of: Optional[Callable[[int, int, int], "np.ndarray"]] = None
+    # block table and lengths of a prompt's sequences, for layers that read the pages (built when one asks)
+    page_source: Optional[Callable[[], Tuple[torch.Tensor, torch.Tensor]]] = None
     # context parallelism: this rank holds one chunk of every sequence; K/V are gathered over cp_group
     cp_group: Any = None
     extras: Dict[str, Any] = field(default_factory=dict)
+
+    def pages(self) -> Tuple[torch.Tensor, torch.Tensor]:
+        """(block table, lengths after this step) of the step's sequences."""
+        if self.block_table is None:
+            self.block_table, self.seq_lens = self.page_source()
+        return self.block_table, self.seq_lens
 
     def visible_context(self, window: Optional[int]) -> Tuple[Optional[torch.Tensor], torch.Tensor]:
         """(flat cache slots of every key the step's tokens can see, packed by sequence; their offsets [B + 1]).  The

@@ -4,9 +4,10 @@ The reference keeps Python lists of per-layer block objects and concatenates the
 (model/core/cache.py:535-868, read path :824-835); its unified manager is lossy by default (H2O,
 quantisation, eviction; cache.py:1886-2038).  Here the cache is two device tensors per layer
 ``[num_blocks, block_size, n_kv_head, head_dim]`` plus an int32 block table per sequence; the decode kernel
-reads pages in place.  ``YvPagedLatentCache`` keeps the same pages, tables and free list with one latent row per token
-and layer instead of keys and values, and gives pages back once every layer's window has passed them.  The cache is exact; eviction policies (LRU of whole sequences, sliding window)
-are opt-in helpers that only edit block tables.
+reads pages in place.  ``YvPagedLayeredCache`` keeps the same pages, tables and free list for layer runs that each store
+what they need (keys and values of sizes of their own, or one latent row per token), and gives pages back once every
+layer's window has passed them.  The cache is exact; eviction policies (LRU of whole sequences, sliding window) are
+opt-in helpers that only edit block tables.
 """
 from __future__ import annotations
 
@@ -161,7 +162,7 @@ class YvPagedKVCache:
     # ---- checkpoint / restore (reference cache.py:2394-2430) ------------------------------------------------
     def state(self) -> Dict[str, object]:
         return {"tables": {k: list(v) for k, v in self.tables.items()}, "lengths": dict(self.lengths),
-                "k": [t.cpu() for t in self.k], "v": [t.cpu() for t in self.v]}
+                "k": [t.cpu() for t in self.k], "v": [None if t is None else t.cpu() for t in self.v]}
 
     def load_state(self, st: Dict[str, object]) -> None:
         self.tables = {int(k): list(v) for k, v in st["tables"].items()}      # type: ignore[union-attr]
@@ -172,37 +173,53 @@ class YvPagedKVCache:
         self.alloc.refs = {b: sum(b in t for t in self.tables.values()) for b in used}
         for mine, saved in ((self.k, st["k"]), (self.v, st["v"])):
             for t, src in zip(mine, saved):                                    # type: ignore[arg-type]
-                t.copy_(src)
+                if t is not None:
+                    t.copy_(src)
 
 
-class YvPagedLatentCache(YvPagedKVCache):
-    """Pages of latent rows: layer i stores ``row_sizes[i]`` numbers per token, ``[num_blocks, block_size, row]``."""
+class YvPagedLayeredCache(YvPagedKVCache):
+    """Pages whose contents differ from layer run to layer run.  Layout i is ``{"row": n}`` (one row of n numbers per
+    token) or ``{"heads": g, "dim": d, "vdim": e}`` (keys ``[num_blocks, block_size, g, d]`` and values ``[.., g, e]``)."""
 
-    def __init__(self, row_sizes: List[int], cfg: YvCacheConfig, device: torch.device, reach: Optional[int] = None):
+    def __init__(self, layouts: List[Dict[str, int]], cfg: YvCacheConfig, device: torch.device, reach: Optional[int] = None):
         self.cfg, self.device = cfg, device
-        self.n_layer, self.hk, self.d = len(row_sizes), 1, max(row_sizes)
-        self.k = [torch.zeros(cfg.num_blocks, cfg.block_size, r, dtype=cfg.dtype, device=device) for r in row_sizes]
-        self.v = []
+        self.n_layer = len(layouts)
+        self.hk = max(m.get("heads", 1) for m in layouts)
+        self.d = max(m["row"] if "row" in m else max(m["dim"], m["vdim"]) for m in layouts)
+        page = lambda *tail: torch.zeros(cfg.num_blocks, cfg.block_size, *tail, dtype=cfg.dtype, device=device)
+        self.k = [page(m["row"]) if "row" in m else page(m["heads"], m["dim"]) for m in layouts]
+        self.v = [None if "row" in m else page(m["heads"], m["vdim"]) for m in layouts]
         self.alloc = YvBlockAllocator(cfg.num_blocks)
         self.tables, self.lengths = {}, {}
         self.layer_offset = 0
         self.reach = reach
 
     def rows(self, idx: int) -> torch.Tensor:
+        if self.v[idx - self.layer_offset] is not None:
+            raise TypeError("this layer stores keys and values: use layer()")
         return self.k[idx - self.layer_offset]
 
     def layer(self, idx: int):
-        raise TypeError("a latent cache has no separate keys and values: use rows()")
+        if self.v[idx - self.layer_offset] is None:
+            raise TypeError("this layer stores one row per token: use rows()")
+        return super().layer(idx)
 
     def bytes(self) -> int:
-        return sum(t.numel() * t.element_size() for t in self.k)
+        return sum(t.numel() * t.element_size() for t in self.k + self.v if t is not None)
+
+
+class YvPagedLatentCache(YvPagedLayeredCache):
+    """Pages of latent rows: layer i stores ``row_sizes[i]`` numbers per token, ``[num_blocks, block_size, row]``."""
+
+    def __init__(self, row_sizes: List[int], cfg: YvCacheConfig, device: torch.device, reach: Optional[int] = None):
+        super().__init__([{"row": r} for r in row_sizes], cfg, device, reach)
 
 
 def cache_for_model(cfg, device: torch.device, num_blocks: int, block_size: Optional[int] = None, tp_size: int = 1,
                     n_layer: Optional[int] = None, dtype: torch.dtype = torch.bfloat16) -> YvPagedKVCache:
     cc = YvCacheConfig(block_size=block_size or cfg.kv_cache_block_size, num_blocks=num_blocks, dtype=dtype)
     if cfg.layer_specs:
-        from .registry import latent_cache_layout
-        rows, reach = latent_cache_layout(cfg)
-        return YvPagedLatentCache(rows, cc, device, reach)
+        from .registry import cache_layout
+        layouts, reach = cache_layout(cfg)
+        return YvPagedLayeredCache(layouts, cc, device, reach)
     return YvPagedKVCache(n_layer or cfg.n_layer, cfg.n_kv_head // tp_size, cfg.head_dim, cc, device)

@@ -171,6 +171,7 @@ def _prefill(model, ids: torch.Tensor, cache: YvPagedKVCache, seq_ids: List[int]
         slots += cache.append_slots(s, S) + [-1] * pad
     ctx.cache = cache
     ctx.slot_map = torch.tensor(slots, dtype=torch.int32).to(ids.device)
+    ctx.page_source = lambda: (cache.block_table_tensor(seq_ids), cache.seq_lens_tensor(seq_ids))
     if want is not None and B != 1:
         raise ValueError("wanted places are given for one sequence at a time")
     out = model(input_ids=ids, ctx=ctx, return_logits=False, return_hidden=True)

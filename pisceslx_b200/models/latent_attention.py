@@ -94,11 +94,12 @@ class YvWindowedLatentAttention(nn.Module):
     def _angles(self, ctx: AttnContext, device: torch.device) -> Tuple[torch.Tensor, torch.Tensor]:
         return self.rotary.tables(ctx.max_position or ctx.max_len, device)
 
-    def forward(self, h: torch.Tensor, ctx: AttnContext) -> torch.Tensor:
-        """h [T, hidden] (normed input, packed tokens) -> [T, hidden]."""
+    def forward(self, h: torch.Tensor, ctx: AttnContext, run: Optional[int] = None) -> torch.Tensor:
+        """h [T, hidden] (normed input, packed tokens) -> [T, hidden]; ``run`` names the cache of a layer that runs more
+        than once."""
         cos, sin = self._angles(ctx, h.device)
         y = L.project(h, self.in_proj)
-        cache = ctx.cache.rows(self.layer_idx) if ctx.cache is not None else None
+        cache = ctx.cache.rows(self.layer_idx if run is None else run) if ctx.cache is not None else None
         cq, rows = L.latent_prep(y, self.q_rank, self.kv_rank, self.rot_dim, self.q_norm, self.kv_norm, cos, sin,
                                  ctx.positions, self.eps, cache, ctx.slot_map, want_rows=not ctx.decode)
         gate = y[:, self.gate_col:self.gate_col + self.heads] if self.gated else None

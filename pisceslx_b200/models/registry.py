@@ -18,11 +18,23 @@ def model_class(cfg: Any) -> type:
     return _BUILDERS[cfg.architecture]()
 
 
-def latent_cache_layout(cfg: Any) -> Tuple[List[int], Optional[int]]:
-    """(numbers per token of every layer's cache row, tokens the widest layer reads back or None)."""
-    rows = [s["mixer"]["kv_rank"] + s["mixer"]["rot_dim"] for s in cfg.layer_specs]
-    windows = [s["mixer"]["window"] for s in cfg.layer_specs]
-    return rows, (max(windows) if all(windows) else None)
+def cache_layout(cfg: Any) -> Tuple[List[Dict[str, int]], Optional[int]]:
+    """(what every layer run of a layered model stores per token, tokens the widest layer reads back or None): either
+    ``{"row": numbers}`` or ``{"heads", "dim", "vdim"}`` of keys and values."""
+    layouts, reach = [], []
+    for i, _, _ in cfg.layer_runs():
+        m = cfg.layer_specs[i]["mixer"]
+        if m["kind"] == "latent_attention":
+            layouts.append({"row": m["kv_rank"] + m["rot_dim"]})
+        else:
+            layouts.append({"heads": m["kv_heads"], "dim": m["dim"], "vdim": m["vdim"]})
+        reach.append(m.get("window"))
+    return layouts, (max(reach) if all(reach) else None)
+
+
+def kernel_families(cfg: Any) -> Tuple[str, ...]:
+    """The operator families (``ops.build.FAMILIES``) that serve a model; empty = the whole library."""
+    return tuple(sorted({s["mixer"]["kind"] for s in cfg.layer_specs}))
 
 
 def _yv() -> type:
@@ -37,3 +49,4 @@ def _layered() -> type:
 
 register_model("", _yv)
 register_model("Gebelorn", _layered)
+register_model("Pitolix", _layered)

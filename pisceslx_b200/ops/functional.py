@@ -66,8 +66,8 @@ def _splitk_plan(M: int, N: int, K: int) -> int:
     return slices if slices > 1 else 0
 
 
-def gemm_skinny(x2: torch.Tensor, w: torch.Tensor, bias: Optional[torch.Tensor] = None) -> Optional[torch.Tensor]:
-    """y = x2 @ w.T through the split-K path, or None when the shape does not call for it."""
+def _splitk_setup(x2: torch.Tensor, w: torch.Tensor) -> Optional[Tuple[int, torch.Tensor, torch.Tensor]]:
+    """(slices, workspace, offsets of the slices) of the split-K product, or None when the shape does not call for it."""
     M, K = x2.shape
     N = w.shape[0]
     slices = _splitk_plan(M, N, K)
@@ -85,9 +85,29 @@ def gemm_skinny(x2: torch.Tensor, w: torch.Tensor, bias: Optional[torch.Tensor] 
     if ws is None or ws.numel() < need:
         ws = torch.empty(max(need, 16 * 128 * 8192), dtype=torch.float32, device=dev)
         _SPLITK_WS[dev.index] = ws
-    out = torch.empty(M, N, dtype=_BF16, device=dev)
+    return slices, ws, offs
+
+
+def gemm_skinny(x2: torch.Tensor, w: torch.Tensor, bias: Optional[torch.Tensor] = None) -> Optional[torch.Tensor]:
+    """y = x2 @ w.T through the split-K path, or None when the shape does not call for it."""
+    plan = _splitk_setup(x2, w)
+    if plan is None:
+        return None
+    _, ws, offs = plan
+    out = torch.empty(x2.shape[0], w.shape[0], dtype=_BF16, device=x2.device)
     _k().gemm_splitk(x2, w, ws, offs, bias, out, _st(x2))
     return out
+
+
+def skinny_parts(x2: torch.Tensor, w: torch.Tensor) -> Optional[torch.Tensor]:
+    """The fp32 parts [slices, 128, N] whose sum is x2 @ w.T, or None when the shape does not call for the split-K path.
+    They live in the shared workspace: the next split-K product on the device overwrites them."""
+    plan = _splitk_setup(x2, w)
+    if plan is None:
+        return None
+    slices, ws, offs = plan
+    _k().gemm_splitk(x2, w, ws, offs, None, None, _st(x2))
+    return ws[:slices * 128 * w.shape[0]].view(slices, 128, w.shape[0])
 
 
 class _LinearFn(torch.autograd.Function):

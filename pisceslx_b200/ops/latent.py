@@ -1,10 +1,10 @@
-"""Operators of latent attention and of the fp32 residual stream around normed branches (serving: no autograd).
+"""Operators of latent attention and of the fp32 residual stream of layered models (serving: no autograd).
 
 CUDA tensors run the kernels of ``csrc/latent.cu``, ``csrc/stream.cu`` and the tcgen05 GEMM in bf16, or their
 CUDA-core forms in fp32 (true 32-bit products); CPU tensors run the plain math of ``ops.reference``."""
 from __future__ import annotations
 
-from typing import Optional, Tuple
+from typing import Optional, Sequence, Tuple
 
 import torch
 
@@ -38,6 +38,22 @@ def project(x: torch.Tensor, w: torch.Tensor, out_fp32: bool = False) -> torch.T
         return F_.linear(x, w, out_fp32=out_fp32)
     out = torch.empty(T, N, dtype=torch.float32 if out_fp32 else x.dtype, device=x.device)
     kernels().linear_simt(x.unsqueeze(0), w.unsqueeze(0), out.unsqueeze(0))
+    return out
+
+
+def project_onto(x: torch.Tensor, z: torch.Tensor, w: torch.Tensor) -> Optional[torch.Tensor]:
+    """x += z [T, K] @ w [N, K]^T on the fp32 stream x [T, N].  The tensor-core product adds to x itself; a skinny one
+    is cut along K and returns its fp32 parts [slices, rows, N] for ``stream_add`` to sum (as do products that run on
+    the CUDA cores or the CPU, in one part): None means that x already holds the sum."""
+    if not x.is_cuda:
+        return torch.nn.functional.linear(z, w.to(z.dtype)).float()
+    if z.dtype == _BF16 and _mappable(z, w) and x.shape[1] % 4 == 0:
+        parts = F_.skinny_parts(z, w)
+        if parts is None:
+            kernels().gemm(z, w, x, False, False, True, 0, _st(z))
+        return parts
+    out = torch.empty_like(x)
+    kernels().linear_simt(z.unsqueeze(0), w.unsqueeze(0), out.unsqueeze(0))
     return out
 
 
@@ -78,6 +94,38 @@ def stream_norm(x: torch.Tensor, y: Optional[torch.Tensor], w_y: Optional[torch.
     h = torch.empty(x.shape, dtype=dtype, device=x.device) if want_h else None
     kernels().stream_norm(x, y, rows, w_y, w_h, h, start, eps, _st(x))
     return h
+
+
+def stream_add(x: torch.Tensor, parts: Optional[torch.Tensor], norms: Sequence[torch.Tensor], offset: float, eps: float,
+               dtype: torch.dtype, table: Optional[torch.Tensor] = None, rows: Optional[torch.Tensor] = None,
+               table_scale: float = 1.0, vec: Optional[torch.Tensor] = None, start: bool = False) -> Tuple[torch.Tensor, ...]:
+    """One pass over the fp32 stream ``x`` [T, C], updated in place: ``x += sum(parts) + table_scale * table[rows] + vec``
+    (each optional; ``start``: ``x = ...``).  ``parts`` is [T, C], or [slices, rows >= T, C] to be summed.  Returns
+    ``x / sqrt(mean(x^2) + eps) * (offset + w)`` in ``dtype`` for each of up to two ``norms``."""
+    if not x.is_cuda:
+        new = torch.zeros_like(x) if start else x.clone()
+        if parts is not None:
+            new += parts.float() if parts.dim() == 2 else parts[:, :x.shape[0]].float().sum(0)
+        if table is not None:
+            new += table[rows].float() * table_scale
+        if vec is not None:
+            new += vec.float()
+        x.copy_(new)
+        return tuple(ref.rms_norm(x, offset + w.float(), eps).to(dtype, copy=True) for w in norms)
+    hs = tuple(torch.empty(x.shape, dtype=dtype, device=x.device) for _ in norms)
+    two = len(norms) > 1
+    kernels().stream_add(x, parts, table, rows if table is not None else None, table_scale, vec, start,
+                         norms[0] if norms else None, norms[1] if two else None, offset, eps, hs[0] if norms else None,
+                         hs[1] if two else None, _st(x))
+    return hs
+
+
+def swiglu(gate_up: torch.Tensor, out: torch.Tensor) -> None:
+    """out [T, F] (a column range) = silu(gate) * up of gate_up [T, 2 F] = [gate | up]."""
+    if not gate_up.is_cuda:
+        out.copy_(ref.swiglu(gate_up))
+        return
+    kernels().gated_silu(gate_up, out)
 
 
 def gelu(x: torch.Tensor) -> torch.Tensor:

@@ -123,6 +123,51 @@ def latent_decode(q_lat: torch.Tensor, cache: torch.Tensor, kv_rank: int, block_
     return out
 
 
+def grouped_prep(q, k, v, bias, bias_at, heads, kv_heads, k_pages, v_pages, slots, positions, cos, sin, rot_dims: int,
+                 unit: bool, temperature, eps: float) -> None:
+    """Biases, unit norm, partial rotation and query temperature; queries in place, keys and values to their slots."""
+    T = q.shape[0]
+    qf, kf, vf = q.float(), k.float(), v.float()
+    if bias is not None:
+        qf, kf, vf = (t + bias[a:a + t.shape[1]].float() for t, a in zip((qf, kf, vf), bias_at))
+    qf, kf = qf.view(T, heads, -1), kf.view(T, kv_heads, -1)
+    if unit:
+        qf, kf = (t * torch.rsqrt(t.pow(2).mean(-1, keepdim=True) + eps) for t in (qf, kf))
+    if rot_dims:
+        qf, kf = (apply_rope(t, cos, sin, positions, rot_dims) for t in (qf, kf))
+    if temperature:
+        steps = torch.div(positions + 1, int(temperature["every"]), rounding_mode="floor").float()
+        qf = qf * (1.0 + temperature["coef"] * torch.log(steps + 1.0)).view(T, 1, 1)
+    q.copy_(qf.reshape(T, -1))
+    at = torch.arange(T, device=q.device) if slots is None else slots.long()
+    keep = at >= 0
+    for rows, pages in ((kf.reshape(T, -1), k_pages), (vf, v_pages)):
+        pages.view(-1, rows.shape[1])[at[keep]] = rows[keep].to(pages.dtype)
+
+
+def grouped_attention(q, k, v, table, lens, cu_q, heads: int, scale: float, sink, gate, out) -> None:
+    """Causal grouped-query attention over pages with a softmax sink and a sigmoid gate per head or per number."""
+    block, kv_heads, dim, vdim = k.shape[1], k.shape[2], k.shape[3], v.shape[3]
+    cq = cu_q.tolist()
+    for b in range(len(cq) - 1):
+        nq = cq[b + 1] - cq[b]
+        n = nq if table is None else int(lens[b])
+        pos = torch.arange(n, device=q.device)
+        slots = pos + cq[b] if table is None else table[b].long()[pos // block] * block + pos % block
+        ks, vs = (t.reshape(-1, kv_heads, t.shape[3])[slots].float().repeat_interleave(heads // kv_heads, 1) for t in (k, v))
+        qs = q[cq[b]:cq[b + 1]].float().view(nq, heads, dim)
+        sc = torch.einsum("qhd,khd->hqk", qs, ks) * scale
+        sc = sc.masked_fill(pos[None, :] > (pos[n - nq:])[:, None], float("-inf"))
+        if sink is not None:
+            sc = torch.cat([sc, sink.float().view(heads, 1, 1).expand(-1, nq, 1)], -1)
+        w = torch.softmax(sc, -1)[..., :n]
+        o = torch.einsum("hqk,khd->qhd", w, vs)
+        if gate is not None:
+            g = torch.sigmoid(gate[cq[b]:cq[b + 1]].float())
+            o = o * g.view(nq, heads, -1)
+        out[cq[b]:cq[b + 1]] = o.reshape(nq, heads * vdim).to(out.dtype)
+
+
 def apply_rope3d(x: torch.Tensor, pos_thw: torch.Tensor, sections: Sequence[int], theta: float = 1e4) -> torch.Tensor:
     """x: [T, heads, d]; the head dim is split into (t, h, w) sections, each rotated by its own position."""
     xf = x.float()
