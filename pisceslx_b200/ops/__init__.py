@@ -10,12 +10,11 @@ from __future__ import annotations
 import os
 import threading
 from pathlib import Path
-from typing import Dict, Optional
+from typing import Dict, Optional, Sequence
 
 import torch
 
 _SO = Path(__file__).resolve().parent / "_yv_ops.so"
-_LAYERED_SO = _SO.with_name("_yv_layered.so")
 _lock = threading.Lock()
 _loaded = False
 _status: Dict[int, torch.Tensor] = {}
@@ -39,20 +38,23 @@ def extension_built() -> bool:
     return _SO.exists()
 
 
-def load_extension(build_if_missing: bool = False, layered: bool = False) -> None:
-    """Load ``_yv_ops.so`` (idempotent).  Raises ``RuntimeError`` when it has not been built.  With ``layered`` a
-    process that runs nothing but layered models takes the smaller ``_yv_layered.so`` when the full one is missing."""
+def load_extension(build_if_missing: bool = False, families: Sequence[str] = ()) -> None:
+    """Load ``_yv_ops.so`` (idempotent).  Raises ``RuntimeError`` when it has not been built.  With ``families`` (mixers
+    of layered models) a process that runs nothing else takes their smaller library when the full one is missing."""
     global _loaded
     if _loaded:
         return
     with _lock:
         if _loaded:
             return
-        so = _LAYERED_SO if layered and not _SO.exists() else _SO
+        so = _SO
+        if families and not _SO.exists():
+            from .build import library
+            so = library(families)
         if not so.exists():
             if build_if_missing or os.environ.get("YV_BUILD_ON_IMPORT") == "1":
                 from .build import build
-                build(layered=so == _LAYERED_SO)
+                build(families=() if so == _SO else families)
             else:
                 raise RuntimeError(
                     f"{so} is missing: run `python -m pisceslx_b200.ops.build` (or __graft_entry__.build()) first")

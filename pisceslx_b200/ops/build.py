@@ -12,20 +12,21 @@ import subprocess
 import sys
 from concurrent.futures import ThreadPoolExecutor
 from pathlib import Path
-from typing import List
+from typing import List, Sequence
 
 HERE = Path(__file__).resolve().parent
 CSRC = HERE / "csrc"
 OBJ = HERE / "build"
 SO = HERE / "_yv_ops.so"
-LAYERED_SO = HERE / "_yv_layered.so"
 
 CUDA_SOURCES = ["gemm.cu", "elementwise.cu", "moe.cu", "loss_optim.cu", "attention.cu", "comm.cu", "noalloc.cu", "ssm.cu", "pq_film.cu",
-                "stream.cu", "latent.cu"]
+                "stream.cu", "latent.cu", "grouped.cu"]
 CPP_SOURCES = ["binding.cpp"]
-# the subset that serves layered models (same operators, a library of its own)
-LAYERED_CUDA_SOURCES = ["gemm.cu", "elementwise.cu", "stream.cu", "latent.cu"]
+# Layered models can be served by a library of their own: the products and the stream, and the operators of their mixers.
+FAMILIES = {"latent_attention": ["latent.cu"], "grouped_attention": ["grouped.cu"]}
+LAYERED_CUDA_SOURCES = ["gemm.cu", "stream.cu"]
 LAYERED_CPP_SOURCES = ["binding_layered.cpp"]
+LAYERED_DEFINES = {"gemm.cu": ["-DYV_SERVING_PRODUCTS"]}
 NVCC_FLAGS = ["-gencode", "arch=compute_100a,code=sm_100a", "-lineinfo", "-O3", "-std=c++17",
               "--expt-relaxed-constexpr", "-Xcompiler", "-fPIC", "-diag-suppress", "550"]
 
@@ -70,8 +71,13 @@ def _run(cmd: List[str]) -> None:
         raise RuntimeError(f"build step failed: {cmd[0]} {cmd[-1]}")
 
 
-def build(verbose: bool = False, force: bool = False, layered: bool = False) -> Path:
-    """Compile what has changed and link ``_yv_ops.so`` (``layered``: the subset ``_yv_layered.so``)."""
+def library(families: Sequence[str] = ()) -> Path:
+    """The library that serves layered models of the given mixers, or the whole one."""
+    return HERE / f"_yv_layered_{'_'.join(sorted(families))}.so" if families else SO
+
+
+def build(verbose: bool = False, force: bool = False, families: Sequence[str] = ()) -> Path:
+    """Compile what has changed and link ``_yv_ops.so`` (``families``: the library that serves those alone)."""
     import torch
     from torch.utils import cpp_extension as ce
 
@@ -80,26 +86,32 @@ def build(verbose: bool = False, force: bool = False, layered: bool = False) -> 
     nvcc = os.path.join(_cuda_home(), "bin", "nvcc")
     jobs = []
     objs: List[Path] = []
-    so = LAYERED_SO if layered else SO
-    for name in LAYERED_CUDA_SOURCES if layered else CUDA_SOURCES:
+    so, families = library(families), sorted(families)
+    cuda, cpp, defines, tag = CUDA_SOURCES, CPP_SOURCES, {}, ""
+    if families:
+        cuda = LAYERED_CUDA_SOURCES + [s for f in families for s in FAMILIES[f]]
+        cpp, defines, tag = LAYERED_CPP_SOURCES, dict(LAYERED_DEFINES), "." + "_".join(families)
+        defines["binding_layered.cpp"] = [f"-DYV_FAMILY_{f.upper()}" for f in families]
+    for name in cuda:
         src = CSRC / name
         if not src.exists():
             continue
-        obj = OBJ / (name + ".o")
+        obj = OBJ / (name + (".serving.o" if name in defines else ".o"))
         objs.append(obj)
         if force or _newer(src, obj, headers):
-            jobs.append([nvcc, "-ccbin", _host_cxx()] + NVCC_FLAGS + ["-I", str(CSRC), "-c", str(src), "-o", str(obj)])
+            jobs.append([nvcc, "-ccbin", _host_cxx()] + NVCC_FLAGS + defines.get(name, []) +
+                        ["-I", str(CSRC), "-c", str(src), "-o", str(obj)])
     inc = []
     for p in ce.include_paths("cuda"):
         inc += ["-isystem", p]
     cxx = _host_cxx()
-    for name in LAYERED_CPP_SOURCES if layered else CPP_SOURCES:
+    for name in cpp:
         src = CSRC / name
-        obj = OBJ / (name + ".o")
+        obj = OBJ / (name + tag + ".o")
         objs.append(obj)
         if force or _newer(src, obj, headers):
             jobs.append([cxx, "-O2", "-std=c++17", "-fPIC", "-DTORCH_EXTENSION_NAME=_yv_ops",
-                         f"-D_GLIBCXX_USE_CXX11_ABI={int(torch._C._GLIBCXX_USE_CXX11_ABI)}",
+                         f"-D_GLIBCXX_USE_CXX11_ABI={int(torch._C._GLIBCXX_USE_CXX11_ABI)}"] + defines.get(name, []) + [
                          "-I", str(CSRC), "-I", os.path.join(_cuda_home(), "include")] + inc +
                         ["-c", str(src), "-o", str(obj)])
     if verbose:

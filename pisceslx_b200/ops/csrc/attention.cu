@@ -187,29 +187,27 @@ int launch_paged_decode(const PagedDecodeArgs& a, cudaStream_t stream) {
   const bool use_mma = use_tma && a.d == 128 && a.block == 64 && (G == 1 || G == 2 || G == 4 || G == 8);
   if (use_mma) {
     // tensor-core kernel: keys are the M dimension, the query heads of the group are padded to N = 16
-    PagedDecodeMmaParams pm;
-    pm.p = p;
-    r = make_tmap_3d(&pm.tma_k, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, a.k_cache, 128, static_cast<uint64_t>(a.hk),
-                     static_cast<uint64_t>(slots), 256, static_cast<uint64_t>(a.hk) * 256, 64, 1, 64);
+    PagedDecodeMmaParams pm = {};
+    r = paged_decode_map(&pm.tma_k, a.k_cache, a.d, a.hk, slots);
     if (r != 0) return -40 + r;
-    r = make_tmap_3d(&pm.tma_v, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, a.v_cache, 128, static_cast<uint64_t>(a.hk),
-                     static_cast<uint64_t>(slots), 256, static_cast<uint64_t>(a.hk) * 256, 64, 1, 64);
+    r = paged_decode_map(&pm.tma_v, a.v_cache, a.d, a.hk, slots);
     if (r != 0) return -50 + r;
-    static PerDeviceInt cfg;
-    if (!cfg.cur()) {
-      r = set_smem(paged_decode_mma_kernel<1>, kDmSmem); if (r) return r;
-      r = set_smem(paged_decode_mma_kernel<2>, kDmSmem); if (r) return r;
-      r = set_smem(paged_decode_mma_kernel<4>, kDmSmem); if (r) return r;
-      r = set_smem(paged_decode_mma_kernel<8>, kDmSmem); if (r) return r;
-      cfg.cur() = 1;
-    }
+    pm.q = p.q; pm.q_ld = static_cast<int64_t>(a.hq) * a.d;
+    pm.o = p.o; pm.o_ld = pm.q_ld;
+    pm.partial_o = a.partial_o; pm.partial_ml = a.partial_ml;
+    pm.block_table = a.block_table; pm.seq_lens = a.seq_lens;
+    pm.hq = a.hq; pm.group = G; pm.chunks = 1;
+    pm.dim = a.d; pm.vdim = a.d; pm.max_blocks_per_seq = a.max_blocks_per_seq;
+    pm.splits = a.splits; pm.num_blocks = a.num_blocks;
+    pm.scale_log2 = p.scale_log2;
+    pm.status = a.status;
     switch (G) {
-      case 1: paged_decode_mma_kernel<1><<<grid, kDmThreads, kDmSmem, stream>>>(pm); break;
-      case 2: paged_decode_mma_kernel<2><<<grid, kDmThreads, kDmSmem, stream>>>(pm); break;
-      case 4: paged_decode_mma_kernel<4><<<grid, kDmThreads, kDmSmem, stream>>>(pm); break;
-      default: paged_decode_mma_kernel<8><<<grid, kDmThreads, kDmSmem, stream>>>(pm); break;
+      case 1: r = paged_decode_mma_run<1, 2>(pm, grid, stream); break;
+      case 2: r = paged_decode_mma_run<2, 2>(pm, grid, stream); break;
+      case 4: r = paged_decode_mma_run<4, 2>(pm, grid, stream); break;
+      default: r = paged_decode_mma_run<8, 2>(pm, grid, stream); break;
     }
-    r = 0;
+    if (r != 0 || a.splits == 1) return r;            // with one split the kernel writes the heads itself
   } else if (use_tma) {
     PagedDecodeTmaParams pp;
     pp.p = p;

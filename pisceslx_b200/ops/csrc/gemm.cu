@@ -1,5 +1,6 @@
 // Host launcher of the tcgen05 GEMM: builds the three tensor maps, picks the template instance and
-// launches one persistent CTA per SM.
+// launches one persistent CTA per SM.  With YV_SERVING_PRODUCTS only the instances that layered models serve with are
+// compiled: both operands K-major, bf16, no collectives.
 #include "per_device.h"
 #include "gemm_sm100.cuh"
 #include "tensormap.h"
@@ -34,6 +35,7 @@ int launch_instance(const GemmParams& p, int grid, cudaStream_t stream) {
   return static_cast<int>(cudaGetLastError());
 }
 
+#ifndef YV_SERVING_PRODUCTS
 // The fused tensor-parallel variants exist for A stored [M,K] and bf16 output only.
 template <int BN, int COMM>
 int dispatch_comm(const GemmArgs& a, const GemmParams& p, int grid, cudaStream_t stream) {
@@ -41,12 +43,18 @@ int dispatch_comm(const GemmArgs& a, const GemmParams& p, int grid, cudaStream_t
   return launch_instance<BN, false, false, __nv_bfloat16, COMM>(p, grid, stream);
 }
 
+#endif
+
 template <int BN, typename OutT>
 int dispatch_layout(const GemmArgs& a, const GemmParams& p, int grid, cudaStream_t stream) {
   if (!a.a_mn && !a.b_mn) return launch_instance<BN, false, false, OutT>(p, grid, stream);
+#ifdef YV_SERVING_PRODUCTS
+  return -90;
+#else
   if (!a.a_mn && a.b_mn) return launch_instance<BN, false, true, OutT>(p, grid, stream);
   if (a.a_mn && a.b_mn) return launch_instance<BN, true, true, OutT>(p, grid, stream);
   return launch_instance<BN, true, false, OutT>(p, grid, stream);
+#endif
 }
 
 }  // namespace
@@ -214,6 +222,9 @@ int launch_gemm(const GemmArgs& a, cudaStream_t stream) {
   const int cap = a.max_ctas > 0 ? a.max_ctas : sm_count();
   const int grid = static_cast<int>(tiles < cap ? tiles : cap);
 
+#ifdef YV_SERVING_PRODUCTS
+  if (mx || a.fp8 || a.comm != 0) return -91;
+#else
   if (mx) {
     return bn == 256 ? launch_instance<256, false, false, __nv_bfloat16, 0, 2>(p, grid, stream)
                      : launch_instance<128, false, false, __nv_bfloat16, 0, 2>(p, grid, stream);
@@ -231,12 +242,48 @@ int launch_gemm(const GemmArgs& a, cudaStream_t stream) {
   if (a.comm == 2) {
     return bn == 256 ? dispatch_comm<256, 2>(a, p, grid, stream) : dispatch_comm<128, 2>(a, p, grid, stream);
   }
+#endif
   if (bn == 256) {
     return a.out_fp32 ? dispatch_layout<256, float>(a, p, grid, stream)
                       : dispatch_layout<256, __nv_bfloat16>(a, p, grid, stream);
   }
   return a.out_fp32 ? dispatch_layout<128, float>(a, p, grid, stream)
                     : dispatch_layout<128, __nv_bfloat16>(a, p, grid, stream);
+}
+
+namespace {
+// out[m, n] = sum_s ws[s][m, n] (+ bias[n]); ws is fp32 [slices][m_pad, N]; four columns per thread
+__global__ void splitk_reduce_kernel(const float* __restrict__ ws, const __nv_bfloat16* __restrict__ bias,
+                                     __nv_bfloat16* __restrict__ out, int slices, int M, int m_pad, int N) {
+  const int64_t quads = static_cast<int64_t>(M) * (N >> 2);
+  for (int64_t i = blockIdx.x * static_cast<int64_t>(blockDim.x) + threadIdx.x; i < quads;
+       i += static_cast<int64_t>(gridDim.x) * blockDim.x) {
+    const int64_t m = i / (N >> 2);
+    const int n = static_cast<int>(i - m * (N >> 2)) << 2;
+    float4 acc = make_float4(0.f, 0.f, 0.f, 0.f);
+    for (int s = 0; s < slices; ++s) {
+      const float4 v = *reinterpret_cast<const float4*>(ws + (static_cast<int64_t>(s) * m_pad + m) * N + n);
+      acc.x += v.x; acc.y += v.y; acc.z += v.z; acc.w += v.w;
+    }
+    if (bias != nullptr) {
+      acc.x += __bfloat162float(bias[n]); acc.y += __bfloat162float(bias[n + 1]);
+      acc.z += __bfloat162float(bias[n + 2]); acc.w += __bfloat162float(bias[n + 3]);
+    }
+    __nv_bfloat162* o = reinterpret_cast<__nv_bfloat162*>(out + m * N + n);
+    o[0] = __floats2bfloat162_rn(acc.x, acc.y);
+    o[1] = __floats2bfloat162_rn(acc.z, acc.w);
+  }
+}
+}  // namespace
+
+int launch_splitk_reduce(const float* ws, const void* bias, void* out, int slices, int M, int m_pad, int N,
+                         cudaStream_t stream) {
+  if (M <= 0 || N <= 0) return 0;
+  if ((N & 3) != 0 || slices <= 0 || m_pad < M) return -1;
+  const int64_t blocks = (static_cast<int64_t>(M) * (N >> 2) + 255) / 256, cap = static_cast<int64_t>(sm_count()) * 16;
+  splitk_reduce_kernel<<<static_cast<unsigned>(blocks < cap ? blocks : cap), 256, 0, stream>>>(
+      ws, reinterpret_cast<const __nv_bfloat16*>(bias), reinterpret_cast<__nv_bfloat16*>(out), slices, M, m_pad, N);
+  return static_cast<int>(cudaGetLastError());
 }
 
 }  // namespace yv

@@ -1,48 +1,10 @@
-// Launcher declarations for latent (low-rank key/value) attention and for the fp32 residual stream around it
-// (latent.cu, stream.cu).  `dtype` is 0 for bf16 and 1 for fp32: activations, weights and cache rows of one call
-// share it; the residual stream, the angles, the scores and every norm are fp32 in both.
+// Launcher declarations for latent (low-rank key/value) attention (latent.cu).  `dtype` is 0 for bf16 and 1 for fp32:
+// activations, weights and cache rows of one call share it; the angles, the scores and every norm are fp32 in both.
 #pragma once
 #include <cuda_runtime.h>
 #include <stdint.h>
 
 namespace yv {
-
-// ------------------------------------------------------------------------------------------------
-// stream.cu
-// ------------------------------------------------------------------------------------------------
-struct StreamNormArgs {
-  float* x = nullptr;              // fp32 stream [rows, cols]; read unless `start`, written when y is given
-  const void* y = nullptr;         // branch output [.., cols] (dtype, or fp32 with y_fp32), null = nothing to add
-  const int64_t* y_rows = nullptr; // optional gather: row t of the branch is y[y_rows[t]]
-  int64_t y_num_rows = 0;          // rows of y when gathered
-  const void* w_y = nullptr;       // weight of the norm on the branch
-  const void* w_h = nullptr;       // weight of the norm in front of the next branch; null = h is the plain stream
-  void* h = nullptr;               // dtype [rows, cols], null = not wanted
-  int64_t rows = 0;
-  int cols = 0;
-  int start = 0;                   // 1: the stream starts here, x = rms(y) * w_y
-  int y_fp32 = 0;
-  float eps = 0.f;
-  int dtype = 0;
-  uint32_t* status = nullptr;
-};
-// x (+)= rms(y) * w_y;  h = rms(x) * w_h (or x).  rms(v) = v / sqrt(mean(v^2) + eps)
-int launch_stream_norm(const StreamNormArgs& a, cudaStream_t stream);
-// out = gelu(in) with the error function; n elements
-int launch_gelu(const void* in, void* out, int64_t n, int dtype, cudaStream_t stream);
-// out[t, j] = gelu_tanh(a[t, j]) * table[token[t], offset + j],  j < dim
-int launch_token_gate(const void* a, int64_t a_stride, const void* table, int64_t table_stride, int64_t vocab,
-                      int64_t offset, const int64_t* token, void* out, int64_t rows, int dim, int dtype,
-                      uint32_t* status, cudaStream_t stream);
-// C[g][m][n] = sum_k A[g][m][k] * B[g][n][k] on the CUDA cores with fp32 accumulation: the exact 32-bit product, and
-// the product for operands a tensor map cannot describe.  Strides in elements.
-struct LinearSimtArgs {
-  const void* a = nullptr; const void* b = nullptr; void* c = nullptr;
-  int64_t M = 0, N = 0, K = 0, groups = 1;
-  int64_t lda = 0, ldb = 0, ldc = 0, a_group = 0, b_group = 0, c_group = 0;
-  int dtype = 0, out_fp32 = 0;
-};
-int launch_linear_simt(const LinearSimtArgs& a, cudaStream_t stream);
 
 // ------------------------------------------------------------------------------------------------
 // latent.cu

@@ -1,345 +1,10 @@
-// Prompt attention of latent layers on the tensor cores: causal with a sliding window, packed sequences whose keys may
-// start before their queries (a portion that continues from the cache), a key part shared by the heads, a value size of
-// its own and a per-head sigmoid gate on the output.
-//
-// One CTA per (128-query block, head, sequence), 192 threads, in the roles of attention_fwd.cuh:
-//   warp 0      TMA producer: Q once, then K_j / V_j tiles through two-stage rings.  A K tile is the head's own part
-//               (1 or 2 slabs of 64 columns) followed by the shared rotary part (one slab); columns past a part's width
-//               are zero-filled by the copy, so any multiple of 8 up to the slab width is a valid size
-//   warp 1      MMA issuer: S_j = Q K_j^T (SS) into one of two TMEM buffers, O += P_j V_j (TS)
-//   warps 2..5  softmax: thread r owns query row r; scores, maxima, exponentials and sums are fp32
-// Key tiles start at the first one that any row of the block can see.
-// TMEM columns: [0,128) S0/P0, [128,256) S1/P1, [256, 256 + 64 NBV) O.
+// Prompt attention of latent layers: the portion kernel over reconstructed keys and values in packed rows, with the rotated
+// key part shared by the heads.
 #pragma once
 #include "latent_ops.h"
-#include "per_device.h"
-#include "sm100.cuh"
-#include "tensormap.h"
+#include "portion_attention.cuh"
 
 namespace yv {
-
-struct LatentPrefillParams {
-  CUtensorMap tma_qn;   // 3-D (dim, head, token), box (64, 1, 128)
-  CUtensorMap tma_qr;   // 3-D (rot_dim, head, token)
-  CUtensorMap tma_k;    // 3-D (dim, head, token)
-  CUtensorMap tma_kr;   // 2-D (rot_dim, token)
-  CUtensorMap tma_v;    // 3-D (vdim, head, token)
-  __nv_bfloat16* o;
-  int64_t o_ld;
-  const __nv_bfloat16* gate;
-  int64_t gate_ld;
-  const int* cu_q;
-  const int* cu_k;
-  int dim, rot_dim, vdim, window;
-  float scale_log2;
-  uint32_t* status;
-};
-
-constexpr int kLpThreads = 192;
-constexpr int kLpBlock = 128;
-constexpr uint32_t kLpSlab = kLpBlock * 128;         // 128 rows x 64 columns
-constexpr float kLpMask = -1.0e30f;
-constexpr float kLpRescale = 8.0f;                   // log2 units
-
-template <int NBN, int NBV>
-struct LatentPrefillSmem {
-  static constexpr int kQK = (NBN + 1) * static_cast<int>(kLpSlab);
-  static constexpr int kV = NBV * static_cast<int>(kLpSlab);
-  static constexpr int kTotal = kQK + 2 * (kQK + kV) + 256 + 1024;
-};
-
-__device__ __forceinline__ float fast_exp2(float x) {
-  float y;
-  asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
-  return y;
-}
-
-template <int NBN, int NBV>
-__global__ void __launch_bounds__(kLpThreads, 1) latent_prefill_kernel(const __grid_constant__ LatentPrefillParams p) {
-  using S = LatentPrefillSmem<NBN, NBV>;
-  constexpr int D = NBV * 64;
-  constexpr uint32_t kIdescQK = make_idesc_bf16(128, 128, false, false);
-  constexpr uint32_t kIdescPV = make_idesc_bf16(128, D, false, true);
-  constexpr uint32_t kTmemCols = 512;
-  constexpr uint32_t kOCol = 256;
-
-  extern __shared__ uint8_t lp_raw[];
-  uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(lp_raw) + 1023) & ~uintptr_t(1023));
-  uint8_t* sQ = smem;
-  uint8_t* sK = sQ + S::kQK;
-  uint8_t* sV = sK + 2 * S::kQK;
-  uint64_t* bars = reinterpret_cast<uint64_t*>(sV + 2 * S::kV);
-  uint64_t* q_full = bars;                 // [1]
-  uint64_t* k_full = bars + 1;             // [2]
-  uint64_t* k_empty = bars + 3;            // [2]
-  uint64_t* v_full = bars + 5;             // [2]
-  uint64_t* v_empty = bars + 7;            // [2]
-  uint64_t* s_full = bars + 9;             // [2]
-  uint64_t* p_full = bars + 11;            // [2]
-  uint64_t* o_done = bars + 13;            // [1]
-  uint32_t* tmem_slot = reinterpret_cast<uint32_t*>(bars + 14);
-
-  const int warp = threadIdx.x >> 5;
-  const int lane = threadIdx.x & 31;
-  const int b = blockIdx.z, h = blockIdx.y;
-  const int q_begin = p.cu_q[b], q_len = p.cu_q[b + 1] - q_begin;
-  const int k_begin = p.cu_k[b], k_len = p.cu_k[b + 1] - k_begin;
-  const int n_qblk = (q_len + kLpBlock - 1) / kLpBlock;
-  const int q_blk = n_qblk - 1 - static_cast<int>(blockIdx.x);       // late (longer) blocks first
-  if (q_blk < 0) return;
-  const int q0 = q_blk * kLpBlock;
-  const int shift = k_len - q_len;                                   // key index of query i is i + shift
-  const int last_key = min(q0 + kLpBlock - 1 + shift, k_len - 1);
-  const int first_key = p.window > 0 ? max(q0 + shift - p.window + 1, 0) : 0;
-  const int j0 = first_key / kLpBlock;
-  const int n_kv = last_key < first_key ? 0 : last_key / kLpBlock + 1 - j0;
-
-  if (threadIdx.x == 0) {
-    tma_prefetch_desc(&p.tma_qn);
-    tma_prefetch_desc(&p.tma_qr);
-    tma_prefetch_desc(&p.tma_k);
-    tma_prefetch_desc(&p.tma_kr);
-    tma_prefetch_desc(&p.tma_v);
-    mbar_init(q_full, 1);
-    for (int s = 0; s < 2; ++s) {
-      mbar_init(&k_full[s], 1);
-      mbar_init(&k_empty[s], 1);
-      mbar_init(&v_full[s], 1);
-      mbar_init(&v_empty[s], 1);
-      mbar_init(&s_full[s], 1);
-      mbar_init(&p_full[s], 128);
-    }
-    mbar_init(o_done, 1);
-    fence_barrier_init();
-  }
-  if (warp == 1) {
-    tmem_alloc(tmem_slot, kTmemCols);
-    tmem_relinquish();
-  }
-  tc_fence_before_sync();
-  __syncthreads();
-  tc_fence_after_sync();
-  const uint32_t tmem_base = *tmem_slot;
-
-  if (warp == 0) {
-    // ------------------------------------ producer ------------------------------------------
-    if (elect_one() && n_kv > 0) {
-      mbar_expect_tx(q_full, S::kQK);
-#pragma unroll
-      for (int c = 0; c < NBN; ++c) tma_load_3d(sQ + c * kLpSlab, &p.tma_qn, q_full, c * 64, h, q_begin + q0);
-      tma_load_3d(sQ + NBN * kLpSlab, &p.tma_qr, q_full, 0, h, q_begin + q0);
-      bool ok = true;
-      for (int j = 0; j < n_kv && ok; ++j) {
-        const int s = j & 1;
-        const uint32_t ph = (j >> 1) & 1u;
-        const int row = k_begin + (j0 + j) * kLpBlock;
-        ok = mbar_wait(&k_empty[s], ph ^ 1u, p.status);
-        if (!ok) break;
-        mbar_expect_tx(&k_full[s], S::kQK);
-#pragma unroll
-        for (int c = 0; c < NBN; ++c)
-          tma_load_3d(sK + s * S::kQK + c * kLpSlab, &p.tma_k, &k_full[s], c * 64, h, row);
-        tma_load_2d(sK + s * S::kQK + NBN * kLpSlab, &p.tma_kr, &k_full[s], 0, row);
-        ok = mbar_wait(&v_empty[s], ph ^ 1u, p.status);
-        if (!ok) break;
-        mbar_expect_tx(&v_full[s], S::kV);
-#pragma unroll
-        for (int c = 0; c < NBV; ++c)
-          tma_load_3d(sV + s * S::kV + c * kLpSlab, &p.tma_v, &v_full[s], c * 64, h, row);
-      }
-    }
-  } else if (warp == 1) {
-    // ------------------------------------ MMA issuer ----------------------------------------
-    if (elect_one() && n_kv > 0) {
-      bool ok = mbar_wait(q_full, 0, p.status);
-      const uint32_t aQ = smem_u32(sQ);
-      const int steps_n = (p.dim + 15) / 16, steps_r = (p.rot_dim + 15) / 16;
-      auto issue_qk = [&](int j) -> bool {
-        const int s = j & 1;
-        if (!mbar_wait(&k_full[s], (j >> 1) & 1u, p.status)) return false;
-        tc_fence_after_sync();
-        const uint32_t aK = smem_u32(sK + s * S::kQK);
-        const uint32_t tS = tmem_base + static_cast<uint32_t>(s * 128);
-        for (int kk = 0; kk < steps_n; ++kk) {
-          const uint32_t off = (kk / 4) * kLpSlab + (kk % 4) * 32;
-          tc_mma_f16_ss(tS, make_smem_desc(aQ + off, 16, 1024), make_smem_desc(aK + off, 16, 1024), kIdescQK,
-                        kk != 0 ? 1u : 0u);
-        }
-        for (int kk = 0; kk < steps_r; ++kk) {
-          const uint32_t off = NBN * kLpSlab + kk * 32;
-          tc_mma_f16_ss(tS, make_smem_desc(aQ + off, 16, 1024), make_smem_desc(aK + off, 16, 1024), kIdescQK, 1u);
-        }
-        tc_commit(&k_empty[s]);
-        tc_commit(&s_full[s]);
-        return true;
-      };
-      if (ok) ok = issue_qk(0);
-      for (int j = 0; j < n_kv && ok; ++j) {
-        if (j + 1 < n_kv) {
-          ok = issue_qk(j + 1);
-          if (!ok) break;
-        }
-        const int s = j & 1;
-        ok = mbar_wait(&p_full[s], (j >> 1) & 1u, p.status);
-        if (!ok) break;
-        ok = mbar_wait(&v_full[s], (j >> 1) & 1u, p.status);
-        if (!ok) break;
-        tc_fence_after_sync();
-        const uint32_t aV = smem_u32(sV + s * S::kV);
-        const uint32_t tP = tmem_base + static_cast<uint32_t>(s * 128);
-        const uint32_t tO = tmem_base + kOCol;
-#pragma unroll
-        for (int kk = 0; kk < kLpBlock / 16; ++kk) {
-          tc_mma_f16_ts(tO, tP + kk * 8, make_smem_desc(aV + kk * 2048, kLpSlab, 1024), kIdescPV,
-                        (j | kk) != 0 ? 1u : 0u);
-        }
-        tc_commit(&v_empty[s]);
-        tc_commit(o_done);
-      }
-    }
-  } else {
-    // ------------------------------------ softmax / epilogue --------------------------------
-    const int quarter = warp & 3;
-    const int row = quarter * 32 + lane;
-    const uint32_t lane_off = static_cast<uint32_t>(quarter * 32) << 16;
-    const int q_pos = q0 + row;
-    const int hi = min(q_pos + shift, k_len - 1);                                    // last visible key
-    const int lo = p.window > 0 ? q_pos + shift - p.window + 1 : 0;                  // first visible key
-    float m_used = -1.0e29f;
-    float l_sum = 0.f;
-    bool ok = true;
-    for (int j = 0; j < n_kv && ok; ++j) {
-      ok = mbar_wait(&s_full[j & 1], (j >> 1) & 1u, p.status);
-      ok = __all_sync(0xFFFFFFFFu, ok);                  // the aligned tcgen05 instructions need a converged warp
-      if (!ok) break;
-      tc_fence_after_sync();
-      const uint32_t tS = tmem_base + lane_off + static_cast<uint32_t>((j & 1) * 128);
-      uint32_t sreg[128];
-      {
-        uint32_t(&c0)[32] = *reinterpret_cast<uint32_t(*)[32]>(&sreg[0]);
-        uint32_t(&c1)[32] = *reinterpret_cast<uint32_t(*)[32]>(&sreg[32]);
-        uint32_t(&c2)[32] = *reinterpret_cast<uint32_t(*)[32]>(&sreg[64]);
-        uint32_t(&c3)[32] = *reinterpret_cast<uint32_t(*)[32]>(&sreg[96]);
-        tmem_ld32(tS, c0);
-        tmem_ld32(tS + 32, c1);
-        tmem_ld32(tS + 64, c2);
-        tmem_ld32(tS + 96, c3);
-        tc_wait_ld();
-      }
-      const int kbase = (j0 + j) * kLpBlock;
-      float mx = kLpMask;
-      if (kbase < lo || kbase + kLpBlock - 1 > hi) {
-#pragma unroll
-        for (int i = 0; i < 128; ++i) {
-          if (kbase + i > hi || kbase + i < lo) sreg[i] = 0xFF800000u;               // -inf
-          mx = fmaxf(mx, __uint_as_float(sreg[i]));
-        }
-      } else {
-#pragma unroll
-        for (int i = 0; i < 128; i += 2)
-          mx = fmaxf(mx, fmaxf(__uint_as_float(sreg[i]), __uint_as_float(sreg[i + 1])));
-      }
-      mx = (mx > 0.5f * kLpMask) ? mx * p.scale_log2 : kLpMask;
-      float alpha = 1.f;
-      bool rescale = false;
-      if (mx > m_used + kLpRescale) {                    // lazy: the reference maximum moves in large steps only
-        alpha = fast_exp2(m_used - mx);
-        m_used = mx;
-        rescale = (j > 0);
-      }
-      float2 rs2 = make_float2(0.f, 0.f);
-      uint32_t pk[64];
-      const float2 sc2 = make_float2(p.scale_log2, p.scale_log2);
-      const float2 nm2 = make_float2(-m_used, -m_used);
-#pragma unroll
-      for (int i = 0; i < 64; ++i) {
-        const float2 x = __ffma2_rn(make_float2(__uint_as_float(sreg[2 * i]), __uint_as_float(sreg[2 * i + 1])), sc2, nm2);
-        const uint32_t bits = pack_bf16(fast_exp2(x.x), fast_exp2(x.y));
-        pk[i] = bits;
-        // the sum takes the rounded weights that the tensor core multiplies
-        rs2 = __fadd2_rn(rs2, make_float2(__uint_as_float(bits << 16), __uint_as_float(bits & 0xFFFF0000u)));
-      }
-      l_sum = l_sum * alpha + (rs2.x + rs2.y);
-      if (__any_sync(0xFFFFFFFFu, rescale)) {
-        ok = mbar_wait(o_done, (j - 1) & 1u, p.status);
-        ok = __all_sync(0xFFFFFFFFu, ok);
-        if (!ok) break;
-        tc_fence_after_sync();
-        const uint32_t tO = tmem_base + lane_off + kOCol;
-#pragma unroll
-        for (int c = 0; c < D / 32; ++c) {
-          uint32_t ov[32];
-          tmem_ld32(tO + c * 32, ov);
-          tc_wait_ld();
-#pragma unroll
-          for (int i = 0; i < 32; ++i) ov[i] = __float_as_uint(__uint_as_float(ov[i]) * alpha);
-          tmem_st32(tO + c * 32, ov);
-        }
-      }
-      {
-        uint32_t(&h0)[32] = *reinterpret_cast<uint32_t(*)[32]>(&pk[0]);
-        uint32_t(&h1)[32] = *reinterpret_cast<uint32_t(*)[32]>(&pk[32]);
-        tmem_st32(tS, h0);
-        tmem_st32(tS + 32, h1);
-      }
-      tc_wait_st();
-      tc_fence_before_sync();
-      mbar_arrive(&p_full[j & 1]);
-    }
-    if (ok && n_kv > 0) {
-      ok = mbar_wait(o_done, (n_kv - 1) & 1u, p.status);
-      ok = __all_sync(0xFFFFFFFFu, ok);
-    }
-    if (ok) {
-      tc_fence_after_sync();
-      const bool valid = q_pos < q_len;
-      float f = (l_sum > 0.f) ? 1.f / l_sum : 0.f;
-      if (valid && p.gate != nullptr) {
-        const float z = __bfloat162float(p.gate[static_cast<int64_t>(q_begin + q_pos) * p.gate_ld + h]);
-        f *= 1.f / (1.f + expf(-z));
-      }
-      __nv_bfloat16* orow = p.o + static_cast<int64_t>(q_begin + q_pos) * p.o_ld + static_cast<int64_t>(h) * p.vdim;
-      const uint32_t tO = tmem_base + lane_off + kOCol;
-#pragma unroll
-      for (int c = 0; c < D / 32; ++c) {
-        uint32_t ov[32];
-        if (n_kv > 0) {
-          tmem_ld32(tO + c * 32, ov);
-          tc_wait_ld();
-        } else {
-#pragma unroll
-          for (int i = 0; i < 32; ++i) ov[i] = 0u;
-        }
-        if (valid) {
-#pragma unroll
-          for (int i = 0; i < 4; ++i) {
-            if (c * 32 + i * 8 < p.vdim) {
-              uint4 v;
-              v.x = pack_bf16(__uint_as_float(ov[8 * i + 0]) * f, __uint_as_float(ov[8 * i + 1]) * f);
-              v.y = pack_bf16(__uint_as_float(ov[8 * i + 2]) * f, __uint_as_float(ov[8 * i + 3]) * f);
-              v.z = pack_bf16(__uint_as_float(ov[8 * i + 4]) * f, __uint_as_float(ov[8 * i + 5]) * f);
-              v.w = pack_bf16(__uint_as_float(ov[8 * i + 6]) * f, __uint_as_float(ov[8 * i + 7]) * f);
-              *reinterpret_cast<uint4*>(orow + c * 32 + i * 8) = v;
-            }
-          }
-        }
-      }
-    }
-  }
-
-  tc_fence_before_sync();
-  __syncthreads();
-  if (p.status != nullptr && *reinterpret_cast<volatile uint32_t*>(p.status) != 0u) {
-    // a wait may have run out with copies still in flight: let them land before the memory is released
-    const uint64_t t0 = globaltimer_ns();
-    while (globaltimer_ns() - t0 < 200000ull) { __nanosleep(1000); }
-    __syncthreads();
-  }
-  if (warp == 1) {
-    tc_fence_after_sync();
-    tmem_dealloc(tmem_base, kTmemCols);
-  }
-}
 
 // The tensor-core kernel takes bf16, parts of up to 128 + 64 columns and values of up to 128, all sizes and pitches
 // multiples of 8 elements, and a positive scale (the row maximum is taken before scaling).
@@ -351,49 +16,27 @@ inline bool latent_attn_on_tensor_cores(const LatentAttnArgs& a) {
          mul8(a.v_ld) && mul8(a.kr_ld) && mul8(a.o_ld) && al16(a.q) && al16(a.k) && al16(a.v) && al16(a.kr) && al16(a.o);
 }
 
-template <int NBN, int NBV>
-int latent_prefill_run(const LatentPrefillParams& p, dim3 grid, cudaStream_t stream) {
-  using S = LatentPrefillSmem<NBN, NBV>;
-  static PerDeviceInt configured;
-  if (!configured.cur()) {
-    const cudaError_t e = cudaFuncSetAttribute(latent_prefill_kernel<NBN, NBV>,
-                                               cudaFuncAttributeMaxDynamicSharedMemorySize, S::kTotal);
-    if (e != cudaSuccess) return static_cast<int>(e);
-    configured.cur() = 1;
-  }
-  latent_prefill_kernel<NBN, NBV><<<grid, kLpThreads, S::kTotal, stream>>>(p);
-  return static_cast<int>(cudaGetLastError());
-}
-
 inline int launch_latent_prefill_mma(const LatentAttnArgs& a, cudaStream_t stream) {
-  LatentPrefillParams p;
-  auto head_map = [&](CUtensorMap* m, const void* base, int d, int64_t head_elems, int64_t tokens, int64_t ld) {
-    return make_tmap_3d(m, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, base, static_cast<uint64_t>(d),
-                        static_cast<uint64_t>(a.heads), static_cast<uint64_t>(tokens),
-                        static_cast<uint64_t>(head_elems) * 2, static_cast<uint64_t>(ld) * 2, 64, 1, kLpBlock);
-  };
+  PortionAttnParams p = {};
   const int hd = a.dim + a.rot_dim;
-  int r = head_map(&p.tma_qn, a.q, a.dim, hd, a.Tq, a.q_ld);
+  int r = portion_head_map(&p.tma_qn, a.q, a.dim, a.heads, hd, a.Tq, a.q_ld, kLpBlock);
   if (r != 0) return -10 + r;
-  r = head_map(&p.tma_qr, static_cast<const __nv_bfloat16*>(a.q) + a.dim, a.rot_dim, hd, a.Tq, a.q_ld);
+  r = portion_head_map(&p.tma_qr, static_cast<const __nv_bfloat16*>(a.q) + a.dim, a.rot_dim, a.heads, hd, a.Tq, a.q_ld, kLpBlock);
   if (r != 0) return -20 + r;
-  r = head_map(&p.tma_k, a.k, a.dim, a.dim, a.Tk, a.k_ld);
+  r = portion_head_map(&p.tma_k, a.k, a.dim, a.heads, a.dim, a.Tk, a.k_ld, 64);
   if (r != 0) return -30 + r;
-  r = head_map(&p.tma_v, a.v, a.vdim, a.vdim, a.Tk, a.v_ld);
+  r = portion_head_map(&p.tma_v, a.v, a.vdim, a.heads, a.vdim, a.Tk, a.v_ld, 64);
   if (r != 0) return -40 + r;
   r = make_tmap_2d(&p.tma_kr, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, a.kr, static_cast<uint64_t>(a.rot_dim),
-                   static_cast<uint64_t>(a.Tk), static_cast<uint64_t>(a.kr_ld), 64, kLpBlock);
+                   static_cast<uint64_t>(a.Tk), static_cast<uint64_t>(a.kr_ld), 64, 64);
   if (r != 0) return -50 + r;
   p.o = static_cast<__nv_bfloat16*>(a.o); p.o_ld = a.o_ld;
-  p.gate = static_cast<const __nv_bfloat16*>(a.gate); p.gate_ld = a.gate_ld;
+  p.gate = static_cast<const __nv_bfloat16*>(a.gate); p.gate_ld = a.gate_ld; p.gate_step = 1;
   p.cu_q = a.cu_q; p.cu_k = a.cu_k;
-  p.dim = a.dim; p.rot_dim = a.rot_dim; p.vdim = a.vdim; p.window = a.window;
-  p.scale_log2 = a.scale * 1.4426950408889634f;
+  p.dim = a.dim; p.rot_dim = a.rot_dim; p.vdim = a.vdim; p.window = a.window; p.group = 1;
+  p.scale_log2 = a.scale * kLpLog2e;
   p.status = a.status;
-  dim3 grid(static_cast<unsigned>((a.max_q + kLpBlock - 1) / kLpBlock), static_cast<unsigned>(a.heads),
-            static_cast<unsigned>(a.batch));
-  if (a.dim <= 64) return a.vdim <= 64 ? latent_prefill_run<1, 1>(p, grid, stream) : latent_prefill_run<1, 2>(p, grid, stream);
-  return a.vdim <= 64 ? latent_prefill_run<2, 1>(p, grid, stream) : latent_prefill_run<2, 2>(p, grid, stream);
+  return portion_attn_dispatch<true>(p, a.max_q, a.heads, a.batch, stream);
 }
 
 }  // namespace yv

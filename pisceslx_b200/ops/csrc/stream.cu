@@ -1,12 +1,13 @@
 // The fp32 residual stream around normed branches: the branch norm, the residual add and the norm in front of the
-// next branch in one pass over a row; the exact GELU; the per-layer token gate; and a CUDA-core product that keeps
-// 32 bits (and takes operands of any size and pitch).
+// next branch in one pass over a row, or a plain join (parts of a product, a table row, a vector) in front of one or two
+// norms; the exact GELU, the gated SiLU and the per-layer token gate; and a CUDA-core product that keeps 32 bits (and
+// takes operands of any size and pitch).
 #include <cuda_bf16.h>
 #include <cuda_runtime.h>
 #include <math.h>
 #include <stdint.h>
 
-#include "latent_ops.h"
+#include "stream_ops.h"
 #include "sm100.cuh"
 
 namespace yv {
@@ -174,6 +175,169 @@ int stream_norm_dispatch(const StreamNormArgs& a, cudaStream_t stream) {
   return static_cast<int>(cudaGetLastError());
 }
 
+// One block per row: the joined row in registers (VPT groups of four columns per thread), then up to two norms of it.
+template <typename T, int VPT>
+__global__ void __launch_bounds__(kStreamThreads) stream_add_kernel(const StreamAddArgs p) {
+  __shared__ float red[kStreamThreads / 32];
+  const int64_t row = blockIdx.x;
+  const int nvec = p.cols >> 2;
+  float* xr = p.x + row * p.cols;
+  float v[VPT][4];
+#pragma unroll
+  for (int i = 0; i < VPT; ++i) {
+    const int c = threadIdx.x + i * kStreamThreads;
+    v[i][0] = v[i][1] = v[i][2] = v[i][3] = 0.f;
+    if (!p.start && c < nvec) load4(xr + c * 4, v[i]);
+  }
+#pragma unroll 4
+  for (int s = 0; s < p.num_parts; ++s) {
+    const float* y = p.parts + s * p.part_stride + row * p.cols;
+#pragma unroll
+    for (int i = 0; i < VPT; ++i) {
+      const int c = threadIdx.x + i * kStreamThreads;
+      float f[4] = {0.f, 0.f, 0.f, 0.f};
+      if (c < nvec) load4(y + c * 4, f);
+#pragma unroll
+      for (int j = 0; j < 4; ++j) v[i][j] += f[j];
+    }
+  }
+  const T* extra[2] = {nullptr, static_cast<const T*>(p.vec)};
+  if (p.table != nullptr) {
+    const int64_t id = p.table_rows[row];
+    if (id >= 0 && id < p.table_num_rows) extra[0] = static_cast<const T*>(p.table) + id * p.cols;
+    else if (threadIdx.x == 0 && p.status != nullptr) atomicOr(p.status, kStatusIndexOutOfRange);
+  }
+#pragma unroll
+  for (int e = 0; e < 2; ++e) {
+    if (extra[e] == nullptr) continue;
+    const float scale = e == 0 ? p.table_scale : 1.f;
+#pragma unroll
+    for (int i = 0; i < VPT; ++i) {
+      const int c = threadIdx.x + i * kStreamThreads;
+      float f[4] = {0.f, 0.f, 0.f, 0.f};
+      if (c < nvec) load4(extra[e] + c * 4, f);
+#pragma unroll
+      for (int j = 0; j < 4; ++j) v[i][j] += f[j] * scale;
+    }
+  }
+  if (p.start || p.num_parts > 0 || p.table != nullptr || p.vec != nullptr) {
+#pragma unroll
+    for (int i = 0; i < VPT; ++i) {
+      const int c = threadIdx.x + i * kStreamThreads;
+      if (c < nvec) store4(xr + c * 4, v[i]);
+    }
+  }
+  if (p.h[0] == nullptr) return;
+  float ss = 0.f;
+#pragma unroll
+  for (int i = 0; i < VPT; ++i)
+#pragma unroll
+    for (int j = 0; j < 4; ++j) ss += v[i][j] * v[i][j];
+  const float r = 1.f / sqrtf(block_sum_all(ss, red) / static_cast<float>(p.cols) + p.eps);
+#pragma unroll
+  for (int n = 0; n < 2; ++n) {
+    if (p.h[n] == nullptr) continue;
+    T* h = static_cast<T*>(p.h[n]) + row * p.cols;
+#pragma unroll
+    for (int i = 0; i < VPT; ++i) {
+      const int c = threadIdx.x + i * kStreamThreads;
+      if (c < nvec) {
+        float w[4], o[4];
+        load4(static_cast<const T*>(p.w[n]) + c * 4, w);
+#pragma unroll
+        for (int j = 0; j < 4; ++j) o[j] = v[i][j] * r * (p.offset + w[j]);
+        store4(h + c * 4, o);
+      }
+    }
+  }
+}
+
+// Any row length: scalar accesses, the row is read again for the norms.
+template <typename T>
+__global__ void __launch_bounds__(kStreamThreads) stream_add_any_kernel(const StreamAddArgs p) {
+  __shared__ float red[kStreamThreads / 32];
+  const int64_t row = blockIdx.x;
+  float* xr = p.x + row * p.cols;
+  const T* tab = nullptr;
+  if (p.table != nullptr) {
+    const int64_t id = p.table_rows[row];
+    if (id >= 0 && id < p.table_num_rows) tab = static_cast<const T*>(p.table) + id * p.cols;
+    else if (threadIdx.x == 0 && p.status != nullptr) atomicOr(p.status, kStatusIndexOutOfRange);
+  }
+  float ss = 0.f;
+  for (int c = threadIdx.x; c < p.cols; c += kStreamThreads) {
+    float n = p.start ? 0.f : xr[c];
+    for (int s = 0; s < p.num_parts; ++s) n += p.parts[s * p.part_stride + row * p.cols + c];
+    if (tab != nullptr) n += to_f(tab[c]) * p.table_scale;
+    if (p.vec != nullptr) n += to_f(static_cast<const T*>(p.vec)[c]);
+    xr[c] = n;
+    ss += n * n;
+  }
+  if (p.h[0] == nullptr) return;
+  const float r = 1.f / sqrtf(block_sum_all(ss, red) / static_cast<float>(p.cols) + p.eps);
+  for (int n = 0; n < 2; ++n) {
+    if (p.h[n] == nullptr) continue;
+    T* h = static_cast<T*>(p.h[n]) + row * p.cols;
+    for (int c = threadIdx.x; c < p.cols; c += kStreamThreads)
+      h[c] = from_f<T>(xr[c] * r * (p.offset + to_f(static_cast<const T*>(p.w[n])[c])));
+  }
+}
+
+template <typename T>
+int stream_add_dispatch(const StreamAddArgs& a, cudaStream_t stream) {
+  const unsigned grid = static_cast<unsigned>(a.rows);
+  auto aligned = [](const void* p, int bytes) { return (reinterpret_cast<uintptr_t>(p) % bytes) == 0; };
+  bool vec = (a.cols % 4) == 0 && a.cols <= 8 * 4 * kStreamThreads && aligned(a.x, 16) && aligned(a.parts, 16) &&
+             (a.part_stride % 4) == 0;
+  for (const void* q : {a.table, a.vec, a.w[0], a.w[1], static_cast<const void*>(a.h[0]), static_cast<const void*>(a.h[1])})
+    vec = vec && aligned(q, 4 * sizeof(T));
+  if (!vec) stream_add_any_kernel<T><<<grid, kStreamThreads, 0, stream>>>(a);
+  else if (a.cols <= 4 * kStreamThreads) stream_add_kernel<T, 1><<<grid, kStreamThreads, 0, stream>>>(a);
+  else if (a.cols <= 2 * 4 * kStreamThreads) stream_add_kernel<T, 2><<<grid, kStreamThreads, 0, stream>>>(a);
+  else if (a.cols <= 4 * 4 * kStreamThreads) stream_add_kernel<T, 4><<<grid, kStreamThreads, 0, stream>>>(a);
+  else stream_add_kernel<T, 8><<<grid, kStreamThreads, 0, stream>>>(a);
+  return static_cast<int>(cudaGetLastError());
+}
+
+// out[t, j] = silu(in[t, j]) * in[t, F + j], N elements (8 or 1) per thread
+template <typename T, int N>
+__global__ void __launch_bounds__(256) gated_silu_kernel(const T* __restrict__ in, int64_t in_ld, T* __restrict__ out,
+                                                         int64_t out_ld, int64_t rows, int F) {
+  const int per = F / N;
+  const int64_t i = static_cast<int64_t>(blockIdx.x) * 256 + threadIdx.x;
+  const int64_t t = i / per;
+  if (t >= rows) return;
+  const int j = static_cast<int>(i - t * per) * N;
+  const T* g = in + t * in_ld + j;
+  T* o = out + t * out_ld + j;
+  auto act = [](float z, float u) { return z / (1.f + expf(-z)) * u; };
+  if constexpr (N == 8) {
+    float a[2][4], b[2][4];
+#pragma unroll
+    for (int q = 0; q < 2; ++q) { load4(g + q * 4, a[q]); load4(g + F + q * 4, b[q]); }
+#pragma unroll
+    for (int q = 0; q < 2; ++q) {
+#pragma unroll
+      for (int k = 0; k < 4; ++k) a[q][k] = act(a[q][k], b[q][k]);
+      store4(o + q * 4, a[q]);
+    }
+  } else {
+    o[0] = from_f<T>(act(to_f(g[0]), to_f(g[F])));
+  }
+}
+
+template <typename T>
+int gated_silu_dispatch(const void* in, int64_t in_ld, void* out, int64_t out_ld, int64_t rows, int F, cudaStream_t stream) {
+  auto al = [](const void* p) { return (reinterpret_cast<uintptr_t>(p) % (4 * sizeof(T))) == 0; };
+  const bool vec = (F % 8) == 0 && (in_ld % 4) == 0 && (out_ld % 4) == 0 && al(in) && al(out);
+  const int64_t items = rows * (vec ? F / 8 : F);
+  if ((items + 255) / 256 > 0x7FFFFFFFll) return -1;
+  const unsigned grid = static_cast<unsigned>((items + 255) / 256);
+  if (vec) gated_silu_kernel<T, 8><<<grid, 256, 0, stream>>>(static_cast<const T*>(in), in_ld, static_cast<T*>(out), out_ld, rows, F);
+  else gated_silu_kernel<T, 1><<<grid, 256, 0, stream>>>(static_cast<const T*>(in), in_ld, static_cast<T*>(out), out_ld, rows, F);
+  return static_cast<int>(cudaGetLastError());
+}
+
 __device__ __forceinline__ float gelu_erf(float z) { return 0.5f * z * (1.f + erff(z * 0.7071067811865476f)); }
 __device__ __forceinline__ float gelu_tanh(float z) {
   return 0.5f * z * (1.f + tanhf(0.7978845608028654f * (z + 0.044715f * z * z * z)));
@@ -270,6 +434,22 @@ int launch_stream_norm(const StreamNormArgs& a, cudaStream_t stream) {
   if (a.dtype == 1) return stream_norm_dispatch<float, float>(a, stream);
   return a.y_fp32 ? stream_norm_dispatch<__nv_bfloat16, float>(a, stream)
                   : stream_norm_dispatch<__nv_bfloat16, __nv_bfloat16>(a, stream);
+}
+
+int launch_stream_add(const StreamAddArgs& a, cudaStream_t stream) {
+  if (a.rows <= 0) return 0;
+  if (a.x == nullptr || a.cols <= 0 || (a.num_parts > 0 && a.parts == nullptr) || (a.table != nullptr && a.table_rows == nullptr)) return -1;
+  if (a.rows > 0x7FFFFFFFll || (a.h[0] == nullptr && a.h[1] != nullptr)) return -2;
+  for (int n = 0; n < 2; ++n)
+    if (a.h[n] != nullptr && a.w[n] == nullptr) return -3;
+  return a.dtype == 1 ? stream_add_dispatch<float>(a, stream) : stream_add_dispatch<__nv_bfloat16>(a, stream);
+}
+
+int launch_gated_silu(const void* in, int64_t in_ld, void* out, int64_t out_ld, int64_t rows, int F, int dtype,
+                      cudaStream_t stream) {
+  if (rows <= 0 || F <= 0) return 0;
+  return dtype == 1 ? gated_silu_dispatch<float>(in, in_ld, out, out_ld, rows, F, stream)
+                    : gated_silu_dispatch<__nv_bfloat16>(in, in_ld, out, out_ld, rows, F, stream);
 }
 
 int launch_gelu(const void* in, void* out, int64_t n, int dtype, cudaStream_t stream) {

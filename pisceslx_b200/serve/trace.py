@@ -77,9 +77,11 @@ def main(argv: Optional[List[str]] = None) -> int:
     if not torch.cuda.is_available():
         print("trace_run needs a GPU", file=sys.stderr)
         return 2
-    from ..engine.loader import load_model_for_inference
+    from ..engine.loader import folder_config, load_model_for_inference
+    from ..models.registry import kernel_families
     from ..ops import load_extension
-    load_extension(build_if_missing=True, layered=True)
+    named = folder_config(args.model)
+    load_extension(build_if_missing=True, families=kernel_families(named) if named is not None else ())
     dtype = DTYPES[args.dtype]
     if dtype == torch.float32:
         torch.backends.cuda.matmul.allow_tf32 = torch.backends.cudnn.allow_tf32 = False
