@@ -6,7 +6,7 @@ weights.
 
     python bench.py --gpus N --steps K --warmup W            (N > 1: launched by torch.distributed.run)
     python bench.py --impl reference ...                     (the reference arm)
-    python bench.py --design gebelorn                        (a layered design beside the closest Yv model)
+    python bench.py --design gebelorn|pitolix                (a layered design beside the closest Yv model)
 
 One JSON line is printed by rank 0.  ``value`` is device-timed (CUDA events around exactly K optimizer steps,
 barrier + synchronize on both sides, max over ranks) with the step's inputs already on the device; ``e2e`` is the
@@ -49,7 +49,7 @@ def parse_args():
                     help="routed experts' forward products in block-scaled e4m3 (a labelled fp8 line, never the headline)")
     ap.add_argument("--ref-limit", type=int, default=300, help="seconds given to the reference's full-size attempt")
     ap.add_argument("--no-ref-context", action="store_true", help="skip the reduced-layer context run of the reference")
-    ap.add_argument("--design", default="", choices=["", "gebelorn"],
+    ap.add_argument("--design", default="", choices=["", "gebelorn", "pitolix"],
                     help="instead of the flagship workload: prefill and decode throughput of this layered design beside "
                          "the closest Yv model at equal size (one GPU, one JSON line)")
     ap.add_argument("--design-sizes", default="", help="comma-separated sizes of --design (default: all)")
@@ -224,7 +224,7 @@ def main() -> None:
         return
     if args.design:
         from pisceslx_b200.serve.bench_layered import main as layered_main
-        layered_main(args.steps, max(args.warmup, 3), args.design_sizes, args.design_shares)
+        layered_main(args.design, args.steps, max(args.warmup, 3), args.design_sizes, args.design_shares)
         return
     os.environ.setdefault("PYTORCH_CUDA_ALLOC_CONF", "expandable_segments:True")
     import torch

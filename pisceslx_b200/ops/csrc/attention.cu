@@ -184,7 +184,7 @@ int launch_paged_decode(const PagedDecodeArgs& a, cudaStream_t stream) {
   // TMA-fed kernel: whole cache blocks of up to 128 tokens travel as one bulk copy each
   const int64_t slots = static_cast<int64_t>(a.num_blocks) * a.block;
   const bool use_tma = a.block >= 16 && a.block <= 128 && a.block % 16 == 0 && slots < (1ll << 31) && !a.force_direct;
-  const bool use_mma = use_tma && a.d == 128 && a.block == 64 && (G == 1 || G == 2 || G == 4 || G == 8);
+  const bool use_mma = use_tma && a.block == 64 && (G == 1 || G == 2 || G == 4 || G == 8);
   if (use_mma) {
     // tensor-core kernel: keys are the M dimension, the query heads of the group are padded to N = 16
     PagedDecodeMmaParams pm = {};
@@ -202,10 +202,10 @@ int launch_paged_decode(const PagedDecodeArgs& a, cudaStream_t stream) {
     pm.scale_log2 = p.scale_log2;
     pm.status = a.status;
     switch (G) {
-      case 1: r = paged_decode_mma_run<1, 2>(pm, grid, stream); break;
-      case 2: r = paged_decode_mma_run<2, 2>(pm, grid, stream); break;
-      case 4: r = paged_decode_mma_run<4, 2>(pm, grid, stream); break;
-      default: r = paged_decode_mma_run<8, 2>(pm, grid, stream); break;
+      case 1: r = a.d == 64 ? paged_decode_mma_run<1, 1>(pm, grid, stream) : paged_decode_mma_run<1, 2>(pm, grid, stream); break;
+      case 2: r = a.d == 64 ? paged_decode_mma_run<2, 1>(pm, grid, stream) : paged_decode_mma_run<2, 2>(pm, grid, stream); break;
+      case 4: r = a.d == 64 ? paged_decode_mma_run<4, 1>(pm, grid, stream) : paged_decode_mma_run<4, 2>(pm, grid, stream); break;
+      default: r = a.d == 64 ? paged_decode_mma_run<8, 1>(pm, grid, stream) : paged_decode_mma_run<8, 2>(pm, grid, stream); break;
     }
     if (r != 0 || a.splits == 1) return r;            // with one split the kernel writes the heads itself
   } else if (use_tma) {

@@ -12,15 +12,17 @@
 // one slab the second 64 rows of the V operand are whatever lies behind the slab (the stage's K tile): those lanes of O^T
 // are never read.
 //
-// grid = (kv heads x chunks of G query heads, sequences, splits), 160 threads; three K/V stages, one CTA per SM with
+// grid = (kv heads x chunks of G query heads, sequences, splits), 224 threads; three K/V stages, one CTA per SM with
 // two slabs and two with one:
 //   warps 0..3  softmax: thread t owns key t of the tile (TMEM lane t of S^T) and output dimension t (lane t of O^T);
 //               the reference maximum per head is kept identically by every thread, the running sum per thread
-//   warp 4      one lane issues everything asynchronous: the TMA copies of the K/V ring (a tile is two cache blocks of
-//               64 tokens, 128B swizzle), S^T one tile ahead into one of two TMEM buffers, and the P V product
-// Hand-offs are mbarriers (TMA -> issuer, S^T done -> softmax, P ready -> issuer, P V done -> both).  The softmax warps
-// meet at ONE named barrier per tile, which asks whether any score exceeds its reference maximum by 2^8; maxima are
-// exchanged and O^T is rescaled only then.
+//   warp 4      one lane issues S^T, up to two tiles ahead of the softmax (two TMEM buffers)
+//   warp 5      one lane issues the P V product (two P buffers), which also frees the tile's stage
+//   warp 6      one lane issues the TMA copies of the K/V ring (a tile is two cache blocks of 64 tokens, 128B swizzle)
+// The issuing is spread over three warps because a tile is short: neither a copy that has not landed nor the descriptor
+// arithmetic of one product may hold up the other.  Hand-offs are mbarriers, one per buffer, so that no barrier can run
+// two phases ahead of a waiter.  The softmax warps meet at ONE named barrier per tile, which asks whether any score
+// exceeds its reference maximum by 2^8; maxima are exchanged and O^T is rescaled only then.
 // Output: with one split the normalised heads (with an optional sink in the denominator and an optional sigmoid gate),
 // otherwise an unnormalised partial (max, sum, out) per query head and split, merged by another kernel.
 #pragma once
@@ -54,9 +56,9 @@ struct PagedDecodeMmaParams {
 constexpr int kDmStages = 3;
 constexpr int kDmTileKeys = 128;
 constexpr int kDmBlock = 64;                                // tokens per cache block
-constexpr int kDmThreads = 160;
+constexpr int kDmThreads = 224;
 constexpr int kDmSlab = kDmTileKeys * 128;                  // [128 keys][64 columns] bf16
-constexpr int kDmPBytes = 2 * 16 * 128;                     // P [16 heads][128 keys] as two 64-key slabs
+constexpr int kDmPBytes = 2 * 16 * 128;                     // one P buffer [16 heads][128 keys] as two 64-key slabs
 constexpr float kDmLog2e = 1.4426950408889634f;
 
 template <int NB>
@@ -64,7 +66,7 @@ struct DecodeMmaSmem {
   static constexpr int kTile = NB * kDmSlab;                // K (or V) tile
   static constexpr int kStage = 2 * kTile;                  // V, then K
   static constexpr int kQ = NB * 16 * 128;                  // Qpad [16][64 NB] in slabs of 64 columns
-  static constexpr int kTotal = kDmStages * kStage + kQ + kDmPBytes + 1024;
+  static constexpr int kTotal = kDmStages * kStage + kQ + 2 * kDmPBytes + 1024;
 };
 
 // byte offset of element (row, col) in a K-major 128B-swizzled slab of 64 columns (rows of 128 bytes)
@@ -90,18 +92,24 @@ __device__ __forceinline__ bool softmax_barrier_or(bool v) {
   return any != 0u;
 }
 
+__device__ __forceinline__ float dm_exp2(float x) {
+  float y;
+  asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+  return y;
+}
+
 template <int G, int NB>
-__global__ void __launch_bounds__(kDmThreads, NB == 1 ? 2 : 1) paged_decode_mma_kernel(const __grid_constant__ PagedDecodeMmaParams p) {
+__global__ void __launch_bounds__(kDmThreads, NB == 1 && G < 16 ? 2 : 1) paged_decode_mma_kernel(const __grid_constant__ PagedDecodeMmaParams p) {
   using S = DecodeMmaSmem<NB>;
   constexpr uint32_t kIdescQK = make_idesc_bf16(128, 16, false, false);
   constexpr uint32_t kIdescPV = make_idesc_bf16(128, 16, true, false);
-  constexpr int kTableCap = 2048;
+  constexpr int kTableCap = 512;
   extern __shared__ uint8_t dsm_raw[];
   uint8_t* dsm = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(dsm_raw) + 1023) & ~uintptr_t(1023));
   uint8_t* sQ = dsm + kDmStages * S::kStage;
   uint8_t* sP = sQ + S::kQ;
-  __shared__ uint64_t full_bar[kDmStages];
-  __shared__ uint64_t s_bar[2], pv_bar, p_bar;
+  __shared__ uint64_t full_bar[kDmStages], empty_bar[kDmStages];
+  __shared__ uint64_t s_bar[2], pv_bar[2], p_bar[2];
   __shared__ uint32_t tmem_slot;
   __shared__ float s_red[4][G];
   __shared__ int s_table[kTableCap];
@@ -109,7 +117,8 @@ __global__ void __launch_bounds__(kDmThreads, NB == 1 ? 2 : 1) paged_decode_mma_
   const int kvh = blockIdx.x / p.chunks, chunk = blockIdx.x % p.chunks, b = blockIdx.y, split = blockIdx.z;
   const int h0 = kvh * p.group + chunk * G;                               // first query head of this CTA
   const int heads = min(G, p.group - chunk * G);
-  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+  const int tid = threadIdx.x, lane = tid & 31;
+  const int warp = __shfl_sync(0xFFFFFFFFu, tid >> 5, 0);                 // known to be uniform
   int seq_len = p.seq_lens[b];
   if (seq_len < 0 || seq_len > static_cast<int64_t>(p.max_blocks_per_seq) * kDmBlock) {   // reported and cut to the row
     if (tid == 0 && p.status != nullptr) atomicOr(p.status, kStatusIndexOutOfRange);
@@ -131,11 +140,8 @@ __global__ void __launch_bounds__(kDmThreads, NB == 1 ? 2 : 1) paged_decode_mma_
   if (tid == 0) {
     tma_prefetch_desc(&p.tma_k);
     tma_prefetch_desc(&p.tma_v);
-    for (int s = 0; s < kDmStages; ++s) mbar_init(&full_bar[s], 1);
-    mbar_init(&s_bar[0], 1);
-    mbar_init(&s_bar[1], 1);
-    mbar_init(&pv_bar, 1);
-    mbar_init(&p_bar, 128);
+    for (int s = 0; s < kDmStages; ++s) { mbar_init(&full_bar[s], 1); mbar_init(&empty_bar[s], 1); }
+    for (int i = 0; i < 2; ++i) { mbar_init(&s_bar[i], 1); mbar_init(&pv_bar[i], 1); mbar_init(&p_bar[i], 128); }
     fence_barrier_init();
   }
   if (warp == 0) {
@@ -150,7 +156,7 @@ __global__ void __launch_bounds__(kDmThreads, NB == 1 ? 2 : 1) paged_decode_mma_
       val = *reinterpret_cast<const uint4*>(p.q + b * p.q_ld + static_cast<int64_t>(h0 + g) * p.dim + col);
     *reinterpret_cast<uint4*>(sQ + c * 2048 + g * 128 + ((v ^ (g & 7)) << 4)) = val;
   }
-  for (int i = tid; i < kDmPBytes / 16; i += kDmThreads) reinterpret_cast<uint4*>(sP)[i] = make_uint4(0, 0, 0, 0);
+  for (int i = tid; i < 2 * kDmPBytes / 16; i += kDmThreads) reinterpret_cast<uint4*>(sP)[i] = make_uint4(0, 0, 0, 0);
   fence_proxy_async_smem();
   tc_fence_before_sync();
   __syncthreads();
@@ -162,72 +168,90 @@ __global__ void __launch_bounds__(kDmThreads, NB == 1 ? 2 : 1) paged_decode_mma_
   // half of the tile is treated as empty
   auto block_ok = [&](int blk) { const int ph = table[blk]; return ph >= 0 && ph < p.num_blocks; };
 
-  if (warp == 4) {
-    // ------------------------------------ issuer ---------------------------------------------
-    if (lane == 0 && n_tiles > 0) {
-      const int slabs_k = (p.dim + 63) / 64, slabs_v = (p.vdim + 63) / 64, steps = (p.dim + 15) / 16;
-      auto issue_tma = [&](int j) {
-        const int s = j % kDmStages;
+  // descriptors differ in their address field only (the low word): base + byte offset / 16
+  const uint32_t hi_desc = static_cast<uint32_t>(make_smem_desc(0, 16, 1024) >> 32);
+  const uint32_t lo_k = static_cast<uint32_t>(make_smem_desc(0, 16, 1024)), lo_mn = static_cast<uint32_t>(make_smem_desc(0, kDmSlab, 1024));
+  auto desc = [&](uint32_t lo) { return (static_cast<uint64_t>(hi_desc) << 32) | lo; };
+  const uint32_t stage0 = smem_u32(dsm) >> 4;
+
+  if (warp == 6) {
+    // ------------------------------------ TMA producer ---------------------------------------
+    if (elect_one()) {
+      const int slabs_k = (p.dim + 63) / 64, slabs_v = (p.vdim + 63) / 64;
+      int s = 0;
+      for (int j = 0; j < n_tiles; ++j) {
+        if (j >= kDmStages && !mbar_wait(&empty_bar[s], (j / kDmStages - 1) & 1u, p.status)) break;
         uint8_t* sv = dsm + static_cast<size_t>(s) * S::kStage;
         uint8_t* sk = sv + S::kTile;
-        uint32_t bytes = 0;
-        for (int h = 0; h < 2; ++h) {
-          const int blk = blk0 + 2 * j + h;
-          if (blk < blk1 && block_ok(blk)) bytes += static_cast<uint32_t>(slabs_k + slabs_v) * (kDmSlab / 2);
-        }
-        if (bytes == 0) {
-          if (p.status != nullptr) atomicOr(p.status, kStatusIndexOutOfRange);
-          mbar_arrive(&full_bar[s]);
-          return;
-        }
-        mbar_expect_tx(&full_bar[s], bytes);
-        for (int h = 0; h < 2; ++h) {
-          const int blk = blk0 + 2 * j + h;
-          if (blk >= blk1) continue;
-          if (!block_ok(blk)) { if (p.status != nullptr) atomicOr(p.status, kStatusIndexOutOfRange); continue; }
-          const int slot = table[blk] * kDmBlock;
-          for (int c = 0; c < slabs_k; ++c) tma_load_3d(sk + c * kDmSlab + h * (kDmSlab / 2), &p.tma_k, &full_bar[s], c * 64, kvh, slot);
-          for (int c = 0; c < slabs_v; ++c) tma_load_3d(sv + c * kDmSlab + h * (kDmSlab / 2), &p.tma_v, &full_bar[s], c * 64, kvh, slot);
-        }
-      };
-      // S^T(j) = K_j Qpad^T into buffer j & 1
-      auto issue_qk = [&](int j) -> bool {
-        const int s = j % kDmStages;
-        if (!mbar_wait(&full_bar[s], (j / kDmStages) & 1u, p.status)) return false;
-        tc_fence_after_sync();
-        const uint32_t aK = smem_u32(dsm + static_cast<size_t>(s) * S::kStage + S::kTile), aQ = smem_u32(sQ);
-        const uint32_t dS = tS + static_cast<uint32_t>((j & 1) * 16);
-        for (int kk = 0; kk < steps; ++kk) {
-          tc_mma_f16_ss(dS, make_smem_desc(aK + (kk / 4) * kDmSlab + (kk % 4) * 32, 16, 1024),
-                        make_smem_desc(aQ + (kk / 4) * 2048 + (kk % 4) * 32, 16, 1024), kIdescQK, kk != 0 ? 1u : 0u);
-        }
-        tc_commit(&s_bar[j & 1]);
-        return true;
-      };
-      const int pre = n_tiles < kDmStages ? n_tiles : kDmStages;
-      for (int j = 0; j < pre; ++j) issue_tma(j);
-      bool iok = issue_qk(0);
-      for (int j = 0; j < n_tiles && iok; ++j) {
-        // S^T of the next tile runs under this tile's softmax; its buffer was last read for tile j - 1, whose
-        // "P ready" this thread has already waited for
-        if (j + 1 < n_tiles) iok = issue_qk(j + 1);
-        if (!iok) break;
-        iok = mbar_wait(&p_bar, j & 1u, p.status);                 // P(j), the V fix-ups and all reads of S^T(j) are done
-        if (!iok) break;
-        tc_fence_after_sync();
-        const uint32_t aV = smem_u32(dsm + static_cast<size_t>(j % kDmStages) * S::kStage);
-        const uint32_t aP = smem_u32(sP);
+        int slot[2];
+        uint32_t halves = 0;
 #pragma unroll
-        for (int kk = 0; kk < kDmTileKeys / 16; ++kk) {
-          tc_mma_f16_ss(tO, make_smem_desc(aV + kk * 2048, kDmSlab, 1024),
-                        make_smem_desc(aP + (kk / 4) * 2048 + (kk % 4) * 32, 16, 1024), kIdescPV,
+        for (int h = 0; h < 2; ++h) {
+          const int blk = blk0 + 2 * j + h;
+          slot[h] = -1;
+          if (blk < blk1) {
+            if (block_ok(blk)) { slot[h] = table[blk] * kDmBlock; ++halves; }
+            else if (p.status != nullptr) atomicOr(p.status, kStatusIndexOutOfRange);
+          }
+        }
+        if (halves == 0) {
+          mbar_arrive(&full_bar[s]);
+        } else {
+          mbar_expect_tx(&full_bar[s], halves * static_cast<uint32_t>(slabs_k + slabs_v) * (kDmSlab / 2));
+#pragma unroll
+          for (int c = 0; c < NB; ++c)
+#pragma unroll
+            for (int h = 0; h < 2; ++h)
+              if (slot[h] >= 0 && c < slabs_k) tma_load_3d(sk + c * kDmSlab + h * (kDmSlab / 2), &p.tma_k, &full_bar[s], c * 64, kvh, slot[h]);
+#pragma unroll
+          for (int c = 0; c < NB; ++c)
+#pragma unroll
+            for (int h = 0; h < 2; ++h)
+              if (slot[h] >= 0 && c < slabs_v) tma_load_3d(sv + c * kDmSlab + h * (kDmSlab / 2), &p.tma_v, &full_bar[s], c * 64, kvh, slot[h]);
+        }
+        if (++s == kDmStages) s = 0;
+      }
+    }
+  } else if (warp == 4) {
+    // ------------------------------------ S^T issuer -----------------------------------------
+    if (elect_one()) {
+      const int steps = (p.dim + 15) / 16;
+      const uint32_t dQ = lo_k + (smem_u32(sQ) >> 4);
+      int s = 0;
+      for (int j = 0; j < n_tiles; ++j) {
+        // the buffer was last read for tile j - 2, whose weights have been reported
+        if (j >= 2 && !mbar_wait(&p_bar[j & 1], ((j - 2) >> 1) & 1u, p.status)) break;
+        if (!mbar_wait(&full_bar[s], (j / kDmStages) & 1u, p.status)) break;
+        tc_fence_after_sync();
+        const uint32_t dK = lo_k + stage0 + static_cast<uint32_t>((s * S::kStage + S::kTile) >> 4);
+        const uint32_t dS = tS + static_cast<uint32_t>((j & 1) * 16);
+#pragma unroll
+        for (int kk = 0; kk < NB * 4; ++kk)
+          if (kk < steps)
+            tc_mma_f16_ss(dS, desc(dK + ((kk / 4) * kDmSlab + (kk % 4) * 32) / 16), desc(dQ + ((kk / 4) * 2048 + (kk % 4) * 32) / 16),
+                          kIdescQK, kk != 0 ? 1u : 0u);
+        tc_commit(&s_bar[j & 1]);
+        if (++s == kDmStages) s = 0;
+      }
+    }
+  } else if (warp == 5) {
+    // ------------------------------------ P V issuer -----------------------------------------
+    if (elect_one()) {
+      const uint32_t dP0 = lo_k + (smem_u32(sP) >> 4);
+      int s = 0;
+      for (int j = 0; j < n_tiles; ++j) {
+        if (!mbar_wait(&full_bar[s], (j / kDmStages) & 1u, p.status)) break;
+        if (!mbar_wait(&p_bar[j & 1], (j >> 1) & 1u, p.status)) break;   // P(j), the V fix-ups, all reads of S^T(j)
+        tc_fence_after_sync();
+        const uint32_t dV = lo_mn + stage0 + static_cast<uint32_t>((s * S::kStage) >> 4);
+        const uint32_t dP = dP0 + static_cast<uint32_t>((j & 1) * (kDmPBytes >> 4));
+#pragma unroll
+        for (int kk = 0; kk < kDmTileKeys / 16; ++kk)
+          tc_mma_f16_ss(tO, desc(dV + kk * (2048 / 16)), desc(dP + ((kk / 4) * 2048 + (kk % 4) * 32) / 16), kIdescPV,
                         (j | kk) != 0 ? 1u : 0u);
-        }
-        tc_commit(&pv_bar);
-        if (j + kDmStages < n_tiles) {                             // the stage is free once P V has read it
-          iok = mbar_wait(&pv_bar, j & 1u, p.status);
-          if (iok) issue_tma(j + kDmStages);
-        }
+        tc_commit(&pv_bar[j & 1]);
+        tc_commit(&empty_bar[s]);
+        if (++s == kDmStages) s = 0;
       }
     }
   } else {
@@ -285,34 +309,38 @@ __global__ void __launch_bounds__(kDmThreads, NB == 1 ? 2 : 1) paged_decode_mma_
         for (int g = 0; g < G; ++g) {
           const float mt = fmaxf(fmaxf(s_red[0][g], s_red[1][g]), fmaxf(s_red[2][g], s_red[3][g]));
           const float mn = (mt > m_run[g] + 8.f) ? mt : m_run[g];
-          alpha[g] = exp2f(m_run[g] - mn);
+          alpha[g] = dm_exp2(m_run[g] - mn);
           m_run[g] = mn;
           l_run[g] *= alpha[g];
+        }
+        if (j > 0) {                                 // the previous product must be complete before O is rescaled
+          ok = mbar_wait(&pv_bar[(j - 1) & 1], ((j - 1) >> 1) & 1u, p.status);
+          ok = __all_sync(0xFFFFFFFFu, ok);
+          if (ok) {
+            tc_fence_after_sync();
+            uint32_t o[16];
+            tmem_ld16(tO + lane_off, o);
+            tc_wait_ld();
+#pragma unroll
+            for (int g = 0; g < G; ++g) o[g] = __float_as_uint(__uint_as_float(o[g]) * alpha[g]);
+            tmem_st16(tO + lane_off, o);
+            tc_wait_st();
+          }
         }
       }
       float pj[G];
 #pragma unroll
-      for (int g = 0; g < G; ++g) pj[g] = exp2f(sc[g] - m_run[g]);        // masked keys: exp2(-1e30 - m) = 0
-      // the previous tile's P V product must be complete before O is rescaled and P is overwritten
-      if (j > 0) {
-        ok = mbar_wait(&pv_bar, (j - 1) & 1u, p.status);
+      for (int g = 0; g < G; ++g) pj[g] = dm_exp2(sc[g] - m_run[g]);      // masked keys: exp2(-1e30 - m) = 0
+      if (j >= 2) {                                  // this P buffer was read by the product of tile j - 2
+        ok = ok && mbar_wait(&pv_bar[j & 1], ((j - 2) >> 1) & 1u, p.status);
         ok = __all_sync(0xFFFFFFFFu, ok);
       }
-      if (ok && moves && j > 0) {
-        tc_fence_after_sync();
-        uint32_t o[16];
-        tmem_ld16(tO + lane_off, o);
-        tc_wait_ld();
-#pragma unroll
-        for (int g = 0; g < G; ++g) o[g] = __float_as_uint(__uint_as_float(o[g]) * alpha[g]);
-        tmem_st16(tO + lane_off, o);
-        tc_wait_st();
-      }
       if (ok) {
+        uint8_t* sp = sP + (j & 1) * kDmPBytes;
 #pragma unroll
         for (int g = 0; g < G; ++g) {
           const __nv_bfloat16 pb = __float2bfloat16(pj[g]);
-          *reinterpret_cast<__nv_bfloat16*>(sP + (tid >> 6) * 2048 + sw128_off(g, tid & 63)) = pb;
+          *reinterpret_cast<__nv_bfloat16*>(sp + (tid >> 6) * 2048 + sw128_off(g, tid & 63)) = pb;
           l_run[g] += __bfloat162float(pb);          // the sum uses the rounded value that the tensor core multiplies
         }
         // rows of V that this tile did not fill: key t's row in every slab (0 * NaN would be NaN)
@@ -326,10 +354,10 @@ __global__ void __launch_bounds__(kDmThreads, NB == 1 ? 2 : 1) paged_decode_mma_
       if (ok) {
         fence_proxy_async_smem();
         tc_fence_before_sync();
-        mbar_arrive(&p_bar);
+        mbar_arrive(&p_bar[j & 1]);
       }
     }
-    if (ok && n_tiles > 0) ok = mbar_wait(&pv_bar, (n_tiles - 1) & 1u, p.status);
+    if (ok && n_tiles > 0) ok = mbar_wait(&pv_bar[(n_tiles - 1) & 1], ((n_tiles - 1) >> 1) & 1u, p.status);
     ok = __all_sync(0xFFFFFFFFu, ok);
 #pragma unroll
     for (int g = 0; g < G; ++g) {

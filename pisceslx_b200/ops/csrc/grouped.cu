@@ -92,16 +92,15 @@ __device__ __forceinline__ float query_factor(const GroupedPrepArgs& p, int pos)
   return 1.f + p.temp_coef * logf(static_cast<float>((pos + 1) / p.temp_every) + 1.f);
 }
 
-// Sixteen lanes to a head, eight numbers to a lane (heads of up to 128 numbers; sizes, pitches and half the rotated part
-// multiples of 8).  The other number of a rotated pair sits half / 8 lanes away.
-template <typename T>
+// LANES (8 or 16) lanes to a head of up to 8 LANES numbers, eight numbers to a lane (sizes, pitches and half the rotated
+// part are multiples of 8).  The other number of a rotated pair sits half / 8 lanes away.
+template <typename T, int LANES>
 __global__ void __launch_bounds__(256) grouped_prep_vec_kernel(const GroupedPrepArgs p) {
-  const int units = p.heads + 2 * p.kv_heads;
-  const int64_t i = static_cast<int64_t>(blockIdx.x) * 16 + (threadIdx.x >> 4);
-  const int64_t t = min(i / units, p.T - 1);                    // whole warps stay together for the shuffles
-  const bool real = i < p.T * units;
-  const int u = real ? static_cast<int>(i - t * units) : 0;
-  const int lane = threadIdx.x & 15, c = lane * 8;
+  const int64_t t = blockIdx.x;
+  int u = blockIdx.y * (256 / LANES) + threadIdx.x / LANES;
+  const bool real = u < p.heads + 2 * p.kv_heads;               // whole warps stay together for the shuffles
+  if (!real) u = 0;
+  const int lane = threadIdx.x % LANES, c = lane * 8;
   const bool lead = real && lane == 0;
   const PrepUnit<T> w = prep_unit<T>(p, t, u, lead);
   const bool in = c < w.size;
@@ -120,7 +119,7 @@ __global__ void __launch_bounds__(256) grouped_prep_vec_kernel(const GroupedPrep
 #pragma unroll
     for (int j = 0; j < 8; ++j) ss += f[j] * f[j];
 #pragma unroll
-    for (int o = 8; o > 0; o >>= 1) ss += __shfl_xor_sync(0xFFFFFFFFu, ss, o, 16);
+    for (int o = LANES / 2; o > 0; o >>= 1) ss += __shfl_xor_sync(0xFFFFFFFFu, ss, o, LANES);
     if (!w.is_v) {
       const float r = 1.f / sqrtf(ss / static_cast<float>(w.size) + p.eps);
 #pragma unroll
@@ -130,10 +129,10 @@ __global__ void __launch_bounds__(256) grouped_prep_vec_kernel(const GroupedPrep
   if (p.rot_dims > 0) {
     const int half = p.rot_dims >> 1, step = half >> 3;
     const bool low = c < half, turned = c < p.rot_dims && !w.is_v;
-    const int peer = low ? lane + step : lane - step;
+    const int peer = (low ? lane + step : lane - step) & (LANES - 1);
     float g[8];
 #pragma unroll
-    for (int j = 0; j < 8; ++j) g[j] = __shfl_sync(0xFFFFFFFFu, f[j], peer & 15, 16);
+    for (int j = 0; j < 8; ++j) g[j] = __shfl_sync(0xFFFFFFFFu, f[j], peer, LANES);
     if (turned) {
       const int64_t row = angle_row(p, p.positions[t], lead) + (low ? c : c - half);
       float cs[8], sn[8];
@@ -154,12 +153,11 @@ __global__ void __launch_bounds__(256) grouped_prep_vec_kernel(const GroupedPrep
 // One warp per head, any sizes; a lane owns whole pairs, so queries can be finished in place.
 template <typename T>
 __global__ void __launch_bounds__(256) grouped_prep_kernel(const GroupedPrepArgs p) {
-  const int units = p.heads + 2 * p.kv_heads;
-  const int64_t i = static_cast<int64_t>(blockIdx.x) * 8 + (threadIdx.x >> 5);
-  if (i >= p.T * units) return;
-  const int64_t t = i / units;
+  const int64_t t = blockIdx.x;
+  const int u = blockIdx.y * 8 + (threadIdx.x >> 5);
+  if (u >= p.heads + 2 * p.kv_heads) return;
   const int lane = threadIdx.x & 31;
-  const PrepUnit<T> w = prep_unit<T>(p, t, static_cast<int>(i - t * units), lane == 0);
+  const PrepUnit<T> w = prep_unit<T>(p, t, u, lane == 0);
   auto at = [&](int c) { return to_f(w.src[c]) + (w.bias != nullptr ? to_f(w.bias[c]) : 0.f); };
   float r = 1.f;
   if (p.unit && !w.is_v) {
@@ -357,16 +355,20 @@ int launch_grouped_prep(const GroupedPrepArgs& a, cudaStream_t stream) {
   if (a.heads <= 0 || a.kv_heads <= 0 || a.dim <= 0 || a.vdim <= 0 || a.rot_dims < 0 || (a.rot_dims & 1) || a.rot_dims > a.dim) return -1;
   if (a.rot_dims > 0 && (a.cos_t == nullptr || a.sin_t == nullptr || a.max_pos <= 0)) return -2;
   if (a.temp_every < 0 || a.positions == nullptr) return -3;
-  const int64_t units = a.T * (a.heads + 2 * a.kv_heads);
-  if ((units + 7) / 8 > 0x7FFFFFFFll) return -4;
+  const int units = a.heads + 2 * a.kv_heads;
+  if (a.T > 0x7FFFFFFFll || (units + 7) / 8 > 65535) return -4;
   bool vec = a.dim <= 128 && a.vdim <= 128 && ((a.dim | a.vdim | (a.rot_dims >> 1)) & 7) == 0 &&
              ((a.q_ld | a.k_ld | a.v_ld) & 7) == 0;
   for (const void* p : {static_cast<const void*>(a.q), a.k, a.v, a.bq, a.bk, a.bv, static_cast<const void*>(a.k_pages),
                         static_cast<const void*>(a.v_pages), static_cast<const void*>(a.cos_t), static_cast<const void*>(a.sin_t)})
     vec = vec && al16(p);
-  const unsigned grid = static_cast<unsigned>(vec ? (units + 15) / 16 : (units + 7) / 8);
-  if (vec && a.dtype == 1) grouped_prep_vec_kernel<float><<<grid, 256, 0, stream>>>(a);
-  else if (vec) grouped_prep_vec_kernel<__nv_bfloat16><<<grid, 256, 0, stream>>>(a);
+  const bool narrow = a.dim <= 64 && a.vdim <= 64;
+  const int per_block = vec ? (narrow ? 32 : 16) : 8;
+  const dim3 grid(static_cast<unsigned>(a.T), static_cast<unsigned>((units + per_block - 1) / per_block));
+  if (vec && a.dtype == 1 && narrow) grouped_prep_vec_kernel<float, 8><<<grid, 256, 0, stream>>>(a);
+  else if (vec && a.dtype == 1) grouped_prep_vec_kernel<float, 16><<<grid, 256, 0, stream>>>(a);
+  else if (vec && narrow) grouped_prep_vec_kernel<__nv_bfloat16, 8><<<grid, 256, 0, stream>>>(a);
+  else if (vec) grouped_prep_vec_kernel<__nv_bfloat16, 16><<<grid, 256, 0, stream>>>(a);
   else if (a.dtype == 1) grouped_prep_kernel<float><<<grid, 256, 0, stream>>>(a);
   else grouped_prep_kernel<__nv_bfloat16><<<grid, 256, 0, stream>>>(a);
   return static_cast<int>(cudaGetLastError());

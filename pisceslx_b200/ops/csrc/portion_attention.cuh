@@ -5,16 +5,19 @@
 //   keys and values in cache pages (a block table per sequence) or in packed rows;
 //   a sink per head (a logit that only counts in the denominator); a sigmoid gate on the output, per head or per number
 //
-// One CTA per (128-query block, head, sequence), 192 threads, in the roles of attention_fwd.cuh:
-//   warp 0      TMA producer: Q once, then K_j / V_j tiles of 128 keys through two-stage rings, 64 rows to a copy (a page
-//               is a multiple of 64).  A K tile is the head's own part (NBN slabs of 64 columns), then the shared part
+// One CTA per (head, 128-query block, sequence), 192 threads, in the roles of attention_fwd.cuh:
+//   warp 0      TMA producer: Q once, then K_j / V_j tiles of 128 keys through rings, 64 rows to a copy (a page is a
+//               multiple of 64).  A K tile is the head's own part (NBN slabs of 64 columns), then the shared part
 //               (one slab); columns past a part's width are zero-filled by the copy, so any multiple of 8 up to the slab
 //               width is a valid size
-//   warp 1      MMA issuer: S_j = Q K_j^T (SS) into one of two TMEM buffers, O += P_j V_j (TS)
+//   warp 1      MMA issuer: S_j = Q K_j^T (SS) into a TMEM buffer, O += P_j V_j (TS)
 //   warps 2..5  softmax: thread r owns query row r; scores, maxima, exponentials and sums are fp32.  Value rows past the
 //               end of a sequence are cleared: what a page holds there must not meet a zero weight as 0 * NaN
 // Key tiles start at the first one that any row of the block can see.
-// TMEM columns: [0,128) S0/P0, [128,256) S1/P1, [256, 256 + 64 NBV) O.
+// The fp32 exponentials of a tile take as long as its two products, so the products of one block have to run under the
+// softmax of another.  Without a shared part two CTAs fit an SM and cover each other: one score buffer, and one stage of
+// keys and values where two do not fit.  With it, one CTA per SM issues S_{j+1} ahead into a second score buffer.
+// TMEM columns: kScores buffers of 128 for S / P, then 64 NBV for O.
 #pragma once
 #include "per_device.h"
 #include "sm100.cuh"
@@ -55,7 +58,11 @@ template <int NBN, int NBV, bool SHARED>
 struct PortionAttnSmem {
   static constexpr int kQK = (NBN + (SHARED ? 1 : 0)) * static_cast<int>(kLpSlab);
   static constexpr int kV = NBV * static_cast<int>(kLpSlab);
-  static constexpr int kTotal = kQK + 2 * (kQK + kV) + 256 + 1024;
+  static constexpr int kCtas = SHARED ? 1 : 2;                       // per SM
+  static constexpr int kScores = SHARED ? 2 : 1;                     // score buffers
+  static constexpr int kStages = SHARED || NBN + NBV == 2 ? 2 : 1;   // tiles of K and V
+  static constexpr uint32_t kTmemCols = SHARED ? 512 : 256;
+  static constexpr int kTotal = kQK + kStages * (kQK + kV) + 256 + 1024;
 };
 
 __device__ __forceinline__ float fast_exp2(float x) {
@@ -67,20 +74,22 @@ __device__ __forceinline__ float fast_exp2(float x) {
 __device__ __forceinline__ float lp_sigmoid(float z) { return 1.f / (1.f + expf(-z)); }
 
 template <int NBN, int NBV, bool SHARED>
-__global__ void __launch_bounds__(kLpThreads, 1) portion_attn_kernel(const __grid_constant__ PortionAttnParams p) {
+__global__ void __launch_bounds__(kLpThreads, PortionAttnSmem<NBN, NBV, SHARED>::kCtas)
+portion_attn_kernel(const __grid_constant__ PortionAttnParams p) {
   using S = PortionAttnSmem<NBN, NBV, SHARED>;
   constexpr int D = NBV * 64;
   constexpr uint32_t kIdescQK = make_idesc_bf16(128, 128, false, false);
   constexpr uint32_t kIdescPV = make_idesc_bf16(128, D, false, true);
-  constexpr uint32_t kTmemCols = 512;
-  constexpr uint32_t kOCol = 256;
+  constexpr int kStages = S::kStages, kScores = S::kScores;
+  constexpr uint32_t kTmemCols = S::kTmemCols;
+  constexpr uint32_t kOCol = kScores * 128;
 
   extern __shared__ uint8_t lp_raw[];
   uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(lp_raw) + 1023) & ~uintptr_t(1023));
   uint8_t* sQ = smem;
   uint8_t* sK = sQ + S::kQK;
-  uint8_t* sV = sK + 2 * S::kQK;
-  uint64_t* bars = reinterpret_cast<uint64_t*>(sV + 2 * S::kV);
+  uint8_t* sV = sK + kStages * S::kQK;
+  uint64_t* bars = reinterpret_cast<uint64_t*>(sV + kStages * S::kV);
   uint64_t* q_full = bars;                 // [1]
   uint64_t* k_full = bars + 1;             // [2]
   uint64_t* k_empty = bars + 3;            // [2]
@@ -93,7 +102,7 @@ __global__ void __launch_bounds__(kLpThreads, 1) portion_attn_kernel(const __gri
 
   const int warp = threadIdx.x >> 5;
   const int lane = threadIdx.x & 31;
-  const int b = blockIdx.z, h = blockIdx.y;
+  const int b = blockIdx.z, h = blockIdx.x;
   const int q_begin = p.cu_q[b], q_len = p.cu_q[b + 1] - q_begin;
   const bool paged = p.table != nullptr;
   const int k_begin = paged ? 0 : p.cu_k[b];
@@ -103,7 +112,7 @@ __global__ void __launch_bounds__(kLpThreads, 1) portion_attn_kernel(const __gri
     k_len = 0;
   }
   const int n_qblk = (q_len + kLpBlock - 1) / kLpBlock;
-  const int q_blk = n_qblk - 1 - static_cast<int>(blockIdx.x);       // late (longer) blocks first
+  const int q_blk = n_qblk - 1 - static_cast<int>(blockIdx.y);       // all heads' late (longer) blocks first
   if (q_blk < 0) return;
   const int q0 = q_blk * kLpBlock;
   const int shift = k_len - q_len;                                   // key index of query i is i + shift
@@ -164,8 +173,8 @@ __global__ void __launch_bounds__(kLpThreads, 1) portion_attn_kernel(const __gri
       constexpr uint32_t kHalf = kLpSlab / 2;
       bool ok = true;
       for (int j = 0; j < n_kv && ok; ++j) {
-        const int s = j & 1;
-        const uint32_t ph = (j >> 1) & 1u;
+        const int s = j % kStages;
+        const uint32_t ph = (j / kStages) & 1u;
         const int row[2] = {source((j0 + j) * kLpBlock), source((j0 + j) * kLpBlock + 64)};
         ok = mbar_wait(&k_empty[s], ph ^ 1u, p.status);
         if (!ok) break;
@@ -194,15 +203,19 @@ __global__ void __launch_bounds__(kLpThreads, 1) portion_attn_kernel(const __gri
       const uint32_t aQ = smem_u32(sQ);
       const int steps_n = (p.dim + 15) / 16, steps_r = SHARED ? (p.rot_dim + 15) / 16 : 0;
       auto issue_qk = [&](int j) -> bool {
-        const int s = j & 1;
-        if (!mbar_wait(&k_full[s], (j >> 1) & 1u, p.status)) return false;
+        const int s = j % kStages;
+        if (!mbar_wait(&k_full[s], (j / kStages) & 1u, p.status)) return false;
+        // a single score buffer still holds the weights of tile j - 1
+        if (kScores == 1 && j > 0 && !mbar_wait(o_done, (j - 1) & 1u, p.status)) return false;
         tc_fence_after_sync();
         const uint32_t aK = smem_u32(sK + s * S::kQK);
-        const uint32_t tS = tmem_base + static_cast<uint32_t>(s * 128);
-        for (int kk = 0; kk < steps_n; ++kk) {
+        const uint32_t tS = tmem_base + static_cast<uint32_t>((j % kScores) * 128);
+#pragma unroll
+        for (int kk = 0; kk < NBN * 4; ++kk) {
           const uint32_t off = (kk / 4) * kLpSlab + (kk % 4) * 32;
-          tc_mma_f16_ss(tS, make_smem_desc(aQ + off, 16, 1024), make_smem_desc(aK + off, 16, 1024), kIdescQK,
-                        kk != 0 ? 1u : 0u);
+          if (kk < steps_n)
+            tc_mma_f16_ss(tS, make_smem_desc(aQ + off, 16, 1024), make_smem_desc(aK + off, 16, 1024), kIdescQK,
+                          kk != 0 ? 1u : 0u);
         }
         if constexpr (SHARED) {
           for (int kk = 0; kk < steps_r; ++kk) {
@@ -211,23 +224,23 @@ __global__ void __launch_bounds__(kLpThreads, 1) portion_attn_kernel(const __gri
           }
         }
         tc_commit(&k_empty[s]);
-        tc_commit(&s_full[s]);
+        tc_commit(&s_full[j % kScores]);
         return true;
       };
       if (ok) ok = issue_qk(0);
       for (int j = 0; j < n_kv && ok; ++j) {
-        if (j + 1 < n_kv) {
-          ok = issue_qk(j + 1);
+        if (kScores == 2 ? j + 1 < n_kv : j > 0) {
+          ok = issue_qk(kScores == 2 ? j + 1 : j);
           if (!ok) break;
         }
-        const int s = j & 1;
-        ok = mbar_wait(&p_full[s], (j >> 1) & 1u, p.status);
+        const int s = j % kStages;
+        ok = mbar_wait(&p_full[j % kScores], (j / kScores) & 1u, p.status);
         if (!ok) break;
-        ok = mbar_wait(&v_full[s], (j >> 1) & 1u, p.status);
+        ok = mbar_wait(&v_full[s], (j / kStages) & 1u, p.status);
         if (!ok) break;
         tc_fence_after_sync();
         const uint32_t aV = smem_u32(sV + s * S::kV);
-        const uint32_t tP = tmem_base + static_cast<uint32_t>(s * 128);
+        const uint32_t tP = tmem_base + static_cast<uint32_t>((j % kScores) * 128);
         const uint32_t tO = tmem_base + kOCol;
 #pragma unroll
         for (int kk = 0; kk < kLpBlock / 16; ++kk) {
@@ -250,11 +263,11 @@ __global__ void __launch_bounds__(kLpThreads, 1) portion_attn_kernel(const __gri
     float l_sum = 0.f;
     bool ok = true;
     for (int j = 0; j < n_kv && ok; ++j) {
-      ok = mbar_wait(&s_full[j & 1], (j >> 1) & 1u, p.status);
+      ok = mbar_wait(&s_full[j % kScores], (j / kScores) & 1u, p.status);
       ok = __all_sync(0xFFFFFFFFu, ok);                  // the aligned tcgen05 instructions need a converged warp
       if (!ok) break;
       tc_fence_after_sync();
-      const uint32_t tS = tmem_base + lane_off + static_cast<uint32_t>((j & 1) * 128);
+      const uint32_t tS = tmem_base + lane_off + static_cast<uint32_t>((j % kScores) * 128);
       uint32_t sreg[128];
       {
         uint32_t(&c0)[32] = *reinterpret_cast<uint32_t(*)[32]>(&sreg[0]);
@@ -268,18 +281,16 @@ __global__ void __launch_bounds__(kLpThreads, 1) portion_attn_kernel(const __gri
         tc_wait_ld();
       }
       const int kbase = (j0 + j) * kLpBlock;
-      float mx = kLpMask;
       if (kbase < lo || kbase + kLpBlock - 1 > hi) {
 #pragma unroll
-        for (int i = 0; i < 128; ++i) {
+        for (int i = 0; i < 128; ++i)
           if (kbase + i > hi || kbase + i < lo) sreg[i] = 0xFF800000u;               // -inf
-          mx = fmaxf(mx, __uint_as_float(sreg[i]));
-        }
-      } else {
-#pragma unroll
-        for (int i = 0; i < 128; i += 2)
-          mx = fmaxf(mx, fmaxf(__uint_as_float(sreg[i]), __uint_as_float(sreg[i + 1])));
       }
+      float mx4[4] = {kLpMask, kLpMask, kLpMask, kLpMask};
+#pragma unroll
+      for (int i = 0; i < 128; i += 2)
+        mx4[(i >> 1) & 3] = fmaxf(mx4[(i >> 1) & 3], fmaxf(__uint_as_float(sreg[i]), __uint_as_float(sreg[i + 1])));
+      float mx = fmaxf(fmaxf(mx4[0], mx4[1]), fmaxf(mx4[2], mx4[3]));
       mx = (mx > 0.5f * kLpMask) ? mx * p.scale_log2 : kLpMask;
       float alpha = 1.f;
       bool rescale = false;
@@ -288,19 +299,6 @@ __global__ void __launch_bounds__(kLpThreads, 1) portion_attn_kernel(const __gri
         m_used = mx;
         rescale = (j > 0);
       }
-      float2 rs2 = make_float2(0.f, 0.f);
-      uint32_t pk[64];
-      const float2 sc2 = make_float2(p.scale_log2, p.scale_log2);
-      const float2 nm2 = make_float2(-m_used, -m_used);
-#pragma unroll
-      for (int i = 0; i < 64; ++i) {
-        const float2 x = __ffma2_rn(make_float2(__uint_as_float(sreg[2 * i]), __uint_as_float(sreg[2 * i + 1])), sc2, nm2);
-        const uint32_t bits = pack_bf16(fast_exp2(x.x), fast_exp2(x.y));
-        pk[i] = bits;
-        // the sum takes the rounded weights that the tensor core multiplies
-        rs2 = __fadd2_rn(rs2, make_float2(__uint_as_float(bits << 16), __uint_as_float(bits & 0xFFFF0000u)));
-      }
-      l_sum = l_sum * alpha + (rs2.x + rs2.y);
       if (__any_sync(0xFFFFFFFFu, rescale)) {
         ok = mbar_wait(o_done, (j - 1) & 1u, p.status);
         ok = __all_sync(0xFFFFFFFFu, ok);
@@ -308,30 +306,44 @@ __global__ void __launch_bounds__(kLpThreads, 1) portion_attn_kernel(const __gri
         tc_fence_after_sync();
         const uint32_t tO = tmem_base + lane_off + kOCol;
 #pragma unroll
-        for (int c = 0; c < D / 32; ++c) {
-          uint32_t ov[32];
-          tmem_ld32(tO + c * 32, ov);
+        for (int c = 0; c < D / 16; ++c) {
+          uint32_t ov[16];
+          tmem_ld16(tO + c * 16, ov);
           tc_wait_ld();
 #pragma unroll
-          for (int i = 0; i < 32; ++i) ov[i] = __float_as_uint(__uint_as_float(ov[i]) * alpha);
-          tmem_st32(tO + c * 32, ov);
+          for (int i = 0; i < 16; ++i) ov[i] = __float_as_uint(__uint_as_float(ov[i]) * alpha);
+          tmem_st16(tO + c * 16, ov);
         }
       }
-      {
-        uint32_t(&h0)[32] = *reinterpret_cast<uint32_t(*)[32]>(&pk[0]);
-        uint32_t(&h1)[32] = *reinterpret_cast<uint32_t(*)[32]>(&pk[32]);
-        tmem_st32(tS, h0);
-        tmem_st32(tS + 32, h1);
+      // P overwrites the scores, half a tile at a time
+      float2 rs2[4] = {make_float2(0.f, 0.f), make_float2(0.f, 0.f), make_float2(0.f, 0.f), make_float2(0.f, 0.f)};
+      const float2 sc2 = make_float2(p.scale_log2, p.scale_log2);
+      const float2 nm2 = make_float2(-m_used, -m_used);
+#pragma unroll
+      for (int half = 0; half < 2; ++half) {
+        uint32_t pk[32];
+#pragma unroll
+        for (int i = 0; i < 32; ++i) {
+          const int e = 64 * half + 2 * i;
+          const float2 x = __ffma2_rn(make_float2(__uint_as_float(sreg[e]), __uint_as_float(sreg[e + 1])), sc2, nm2);
+          const uint32_t bits = pack_bf16(fast_exp2(x.x), fast_exp2(x.y));
+          pk[i] = bits;
+          // the sum takes the rounded weights that the tensor core multiplies
+          rs2[i & 3] = __fadd2_rn(rs2[i & 3], make_float2(__uint_as_float(bits << 16), __uint_as_float(bits & 0xFFFF0000u)));
+        }
+        tmem_st32(tS + 32 * half, pk);
       }
+      const float2 rsum = __fadd2_rn(__fadd2_rn(rs2[0], rs2[1]), __fadd2_rn(rs2[2], rs2[3]));
+      l_sum = l_sum * alpha + (rsum.x + rsum.y);
       tc_wait_st();
       if (kbase + kLpBlock > k_len) {                    // the sequence ends in this tile: clear the rows behind it
-        ok = mbar_wait(&v_full[j & 1], (j >> 1) & 1u, p.status);
+        ok = mbar_wait(&v_full[j % kStages], (j / kStages) & 1u, p.status);
         ok = __all_sync(0xFFFFFFFFu, ok);
         if (!ok) break;
         if (kbase + row >= k_len) {
 #pragma unroll
           for (int c = 0; c < NBV; ++c) {
-            uint4* vr = reinterpret_cast<uint4*>(sV + (j & 1) * S::kV + c * kLpSlab + row * 128);
+            uint4* vr = reinterpret_cast<uint4*>(sV + (j % kStages) * S::kV + c * kLpSlab + row * 128);
 #pragma unroll
             for (int i = 0; i < 8; ++i) vr[i] = make_uint4(0, 0, 0, 0);
           }
@@ -339,7 +351,7 @@ __global__ void __launch_bounds__(kLpThreads, 1) portion_attn_kernel(const __gri
         fence_proxy_async_smem();
       }
       tc_fence_before_sync();
-      mbar_arrive(&p_full[j & 1]);
+      mbar_arrive(&p_full[j % kScores]);
     }
     if (ok && n_kv > 0) {
       ok = mbar_wait(o_done, (n_kv - 1) & 1u, p.status);
@@ -427,7 +439,8 @@ int portion_attn_run(const PortionAttnParams& p, dim3 grid, cudaStream_t stream)
 
 template <bool SHARED>
 int portion_attn_dispatch(const PortionAttnParams& p, int max_q, int heads, int batch, cudaStream_t stream) {
-  dim3 grid(static_cast<unsigned>((max_q + kLpBlock - 1) / kLpBlock), static_cast<unsigned>(heads),
+  if ((max_q + kLpBlock - 1) / kLpBlock > 65535) return -3;
+  dim3 grid(static_cast<unsigned>(heads), static_cast<unsigned>((max_q + kLpBlock - 1) / kLpBlock),
             static_cast<unsigned>(batch));
   if (p.dim <= 64)
     return p.vdim <= 64 ? portion_attn_run<1, 1, SHARED>(p, grid, stream) : portion_attn_run<1, 2, SHARED>(p, grid, stream);

@@ -302,12 +302,10 @@ int stream_add_dispatch(const StreamAddArgs& a, cudaStream_t stream) {
 // out[t, j] = silu(in[t, j]) * in[t, F + j], N elements (8 or 1) per thread
 template <typename T, int N>
 __global__ void __launch_bounds__(256) gated_silu_kernel(const T* __restrict__ in, int64_t in_ld, T* __restrict__ out,
-                                                         int64_t out_ld, int64_t rows, int F) {
-  const int per = F / N;
-  const int64_t i = static_cast<int64_t>(blockIdx.x) * 256 + threadIdx.x;
-  const int64_t t = i / per;
-  if (t >= rows) return;
-  const int j = static_cast<int>(i - t * per) * N;
+                                                         int64_t out_ld, int F) {
+  const int64_t t = blockIdx.x;
+  const int j = (blockIdx.y * 256 + threadIdx.x) * N;
+  if (j >= F) return;
   const T* g = in + t * in_ld + j;
   T* o = out + t * out_ld + j;
   auto act = [](float z, float u) { return z / (1.f + expf(-z)) * u; };
@@ -330,11 +328,11 @@ template <typename T>
 int gated_silu_dispatch(const void* in, int64_t in_ld, void* out, int64_t out_ld, int64_t rows, int F, cudaStream_t stream) {
   auto al = [](const void* p) { return (reinterpret_cast<uintptr_t>(p) % (4 * sizeof(T))) == 0; };
   const bool vec = (F % 8) == 0 && (in_ld % 4) == 0 && (out_ld % 4) == 0 && al(in) && al(out);
-  const int64_t items = rows * (vec ? F / 8 : F);
-  if ((items + 255) / 256 > 0x7FFFFFFFll) return -1;
-  const unsigned grid = static_cast<unsigned>((items + 255) / 256);
-  if (vec) gated_silu_kernel<T, 8><<<grid, 256, 0, stream>>>(static_cast<const T*>(in), in_ld, static_cast<T*>(out), out_ld, rows, F);
-  else gated_silu_kernel<T, 1><<<grid, 256, 0, stream>>>(static_cast<const T*>(in), in_ld, static_cast<T*>(out), out_ld, rows, F);
+  const int blocks = ((vec ? F / 8 : F) + 255) / 256;
+  if (rows > 0x7FFFFFFFll || blocks > 65535) return -1;
+  const dim3 grid(static_cast<unsigned>(rows), static_cast<unsigned>(blocks));
+  if (vec) gated_silu_kernel<T, 8><<<grid, 256, 0, stream>>>(static_cast<const T*>(in), in_ld, static_cast<T*>(out), out_ld, F);
+  else gated_silu_kernel<T, 1><<<grid, 256, 0, stream>>>(static_cast<const T*>(in), in_ld, static_cast<T*>(out), out_ld, F);
   return static_cast<int>(cudaGetLastError());
 }
 

@@ -387,6 +387,15 @@ def attention(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, cu_q: torch.Ten
     return o.reshape(-1, hq * d)
 
 
+def paged_splits(units: int, table_width: int, per_sm: int = 1) -> int:
+    """Key ranges per sequence of a paged decode step over ``units`` (sequence, kv head) pairs.  It depends on shapes only
+    (so that a captured step can be replayed): the count that minimises waves of CTAs times tiles of one CTA (two pages
+    each), with three tiles' time for a CTA's start and end and four for joining the ranges."""
+    tiles, room = -(-table_width // 2), 148 * per_sm
+    cost = lambda s: -(-units * s // room) * (-(-tiles // s) + 3) + (4 + 0.1 * s if s > 1 else 0)
+    return min(range(1, min(32, max(tiles, 1)) + 1), key=cost)
+
+
 def paged_decode(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tensor, block_table: torch.Tensor,
                  seq_lens: torch.Tensor, scale: Optional[float] = None, splits: int = 0) -> torch.Tensor:
     """One decode step over the paged cache: q [B,hq,d] -> [B,hq,d] (no autograd)."""
@@ -395,11 +404,7 @@ def paged_decode(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tensor, 
     if not q.is_cuda:
         return ref.paged_decode(q, k_cache, v_cache, block_table, seq_lens, scale)
     if splits <= 0:
-        ctas = B * k_cache.shape[2]
-        # one CTA per SM is resident: aim at four or more waves of CTAs so that the last, partial wave is a small
-        # share of the run, without cutting a sequence into pieces shorter than two 128-key tiles
-        splits = max(1, min(32, -(-(4 * 148) // max(ctas, 1))))
-        splits = min(splits, max(1, block_table.shape[1] // 4))
+        splits = paged_splits(B * k_cache.shape[2], block_table.shape[1], 2 if d <= 64 else 1)
     o = torch.empty_like(q)
     po = torch.empty(B, hq, splits, d, dtype=torch.float32, device=q.device)
     pml = torch.empty(B, hq, splits, 2, dtype=torch.float32, device=q.device)

@@ -10,6 +10,7 @@ from typing import Dict, List, Optional
 import torch
 
 from . import kernels, reference as ref, status_word
+from .functional import paged_splits
 
 
 def _st(t: torch.Tensor) -> torch.Tensor:
@@ -49,14 +50,6 @@ def grouped_attention(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, table: 
     kernels().grouped_attn(q, k, v, table, lens, cu_q, max_q, heads, scale, sink, gate, out, simt, _st(q))
 
 
-def grouped_splits(batch: int, groups: int, table_width: int, per_sm: int = 1) -> int:
-    """Key ranges per sequence of the decode kernel.  It depends on shapes only (so that a captured step can be
-    replayed): enough CTAs for four waves, so that the last, partial one is a small share, but no range shorter than two
-    tiles of 128 keys."""
-    want = max(1, min(32, -(-(4 * 148 * per_sm) // max(batch * groups, 1))))
-    return min(want, max(1, table_width // 4))
-
-
 def grouped_decode(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, table: torch.Tensor, lens: torch.Tensor, heads: int,
                    scale: float, sink: Optional[torch.Tensor], gate: Optional[torch.Tensor], out: torch.Tensor,
                    simt: bool = False, splits: int = 0) -> None:
@@ -68,7 +61,8 @@ def grouped_decode(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, table: tor
         return
     B, kv_heads, vdim = q.shape[0], k.shape[2], v.shape[3]
     if splits <= 0:
-        splits = grouped_splits(B, kv_heads * -(-(heads // kv_heads) // 16), table.shape[1])
+        small = max(q.shape[1] // heads, vdim) <= 64
+        splits = paged_splits(B * kv_heads * -(-(heads // kv_heads) // 16), table.shape[1], 2 if small else 1)
     po = pml = None
     if splits > 1:
         po = torch.empty(B * heads * splits * vdim, dtype=torch.float32, device=q.device)

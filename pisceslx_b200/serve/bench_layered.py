@@ -1,20 +1,24 @@
 """Prefill and decode throughput of a layered design beside the Yv trunk's closest configuration at equal size
-(``bench.py --design gebelorn``).
+(``bench.py --design gebelorn`` or ``pitolix``).
 
-The closest existing model is the Yv trunk with dense feed-forwards and its low-rank attention (``use_mla`` with the
-shared rotary slice): same width, layers, heads, ranks and vocabulary, a SwiGLU feed-forward of the same number of
-parameters, full causal attention (the design's window covers the whole context of the decode case).  Both run random
-weights through the serving engine: a prompt is one ``run_tokens`` call, a decode step one replay of a captured step.
-Times are CUDA events around the calls after three warm-ups; weights and caches are larger than L2."""
+* Gebelorn: the Yv trunk with dense feed-forwards and its low-rank attention (``use_mla`` with the shared rotary slice):
+  same width, layers, heads, ranks and vocabulary, a SwiGLU feed-forward of the same number of parameters, full causal
+  attention (the design's window covers the whole context of the decode case).
+* Pitolix: the Yv trunk with dense SwiGLU feed-forwards and grouped-query attention: same width, query and key/value heads,
+  head size, feed-forward and vocabulary, as many layers as the design has layer runs (two layers are passed twice).
+
+Both run random weights through the serving engine: a prompt is one ``run_tokens`` call, a decode step one replay of a
+captured step.  Times are CUDA events around the calls after three warm-ups; weights and caches are larger than L2."""
 from __future__ import annotations
 
 import json
 import time
-from typing import Any, Dict, List, Tuple
+from typing import Any, Callable, Dict, List, Tuple
 
 import torch
 
-SIZES: Dict[str, Dict[str, int]] = {
+VOCAB = 32000
+GEBELORN_SIZES: Dict[str, Dict[str, int]] = {
     "w1024": dict(width=1024, heads=16, dim=64, rot=32, vdim=64, kv_rank=256, q_rank=512, ff=4096, side=64, window=1024,
                   layers=8, prompt=8192, batch=64, context=4096),
     "w2048": dict(width=2048, heads=16, dim=128, rot=64, vdim=128, kv_rank=512, q_rank=1536, ff=8192, side=256,
@@ -22,10 +26,14 @@ SIZES: Dict[str, Dict[str, int]] = {
     "w4096": dict(width=4096, heads=32, dim=128, rot=64, vdim=128, kv_rank=512, q_rank=1536, ff=16384, side=256,
                   window=4096, layers=4, prompt=8192, batch=64, context=4096),
 }
-VOCAB = 32000
+PITOLIX_SIZES: Dict[str, Dict[str, int]] = {
+    "w1024": dict(width=1024, heads=16, kv_heads=4, dim=64, rot=32, ff=2816, runs=8, prompt=8192, batch=64, context=4096),
+    "w2048": dict(width=2048, heads=16, kv_heads=4, dim=128, rot=64, ff=5632, runs=8, prompt=8192, batch=64, context=4096),
+    "w4096": dict(width=4096, heads=32, kv_heads=8, dim=128, rot=64, ff=11264, runs=5, prompt=8192, batch=64, context=4096),
+}
 
 
-def design_config(s: Dict[str, int]):
+def gebelorn_config(s: Dict[str, int]):
     from ..config import YvConfig
     layer = {"type": "latent_attention",
              "mixer": {"heads": s["heads"], "dim": s["dim"], "rot_dim": s["rot"], "vdim": s["vdim"], "kv_rank": s["kv_rank"],
@@ -37,13 +45,41 @@ def design_config(s: Dict[str, int]):
                                "vocab": VOCAB, "width": s["width"], "token_side": {"dim": s["side"]}})
 
 
-def closest_config(s: Dict[str, int]):
+def gebelorn_closest(s: Dict[str, int]):
     from ..config import YvConfig
     return YvConfig(vocab_size=VOCAB, hidden_size=s["width"], n_layer=s["layers"], n_head=s["heads"], n_kv_head=s["heads"],
                     head_dim=128 if s["dim"] > 64 else 64, intermediate_size=(s["ff"] * 2 // 3 + 63) // 64 * 64,
                     moe_num_experts=0, moe_shared_experts=0, use_mla=True, kv_lora_rank=s["kv_rank"],
                     mla_q_lora_rank=s["q_rank"], mla_rope_dim=s["rot"], use_enhanced_mla=True, tie_word_embeddings=False,
                     max_position_embeddings=16384, use_gradient_checkpointing=False, eos_token_id=-1)
+
+
+def pitolix_config(s: Dict[str, int]):
+    """One layer in three has normed queries and keys, the others rotate; layers 0 and 1 are passed twice."""
+    from ..config import YvConfig
+    base = {"heads": s["heads"], "kv_heads": s["kv_heads"], "dim": s["dim"], "vdim": s["dim"], "scale": s["dim"] ** -0.5}
+    mlp = {"kind": "dense", "ff": s["ff"]}
+    rotated = {"type": "attention_2", "mixer": {**base, "rot": {"dims": s["rot"], "base": 10000.0}}, "mlp": mlp}
+    normed = {"type": "attention", "mixer": {**base, "q_temp": {"coef": 0.2, "every": 1024}}, "mlp": mlp}
+    layers = [normed if i % 3 == 2 else rotated for i in range(s["runs"] - 2)]
+    return YvConfig.from_dict({"architecture": "Pitolix", "layers": layers, "norm": {"eps": 1e-6}, "vocab": VOCAB,
+                               "width": s["width"], "embedding": {"scale": s["width"] ** 0.5},
+                               "loop": {"start": 0, "stop": 2, "times": 2}})
+
+
+def pitolix_closest(s: Dict[str, int]):
+    from ..config import YvConfig
+    return YvConfig(vocab_size=VOCAB, hidden_size=s["width"], n_layer=s["runs"], n_head=s["heads"], n_kv_head=s["kv_heads"],
+                    head_dim=s["dim"], intermediate_size=s["ff"], moe_num_experts=0, moe_shared_experts=0,
+                    tie_word_embeddings=False, max_position_embeddings=16384, use_gradient_checkpointing=False,
+                    eos_token_id=-1)
+
+
+# name -> (sizes, the design's configuration, the closest Yv configuration)
+DESIGNS: Dict[str, Tuple[Dict[str, Dict[str, int]], Callable[..., Any], Callable[..., Any]]] = {
+    "gebelorn": (GEBELORN_SIZES, gebelorn_config, gebelorn_closest),
+    "pitolix": (PITOLIX_SIZES, pitolix_config, pitolix_closest),
+}
 
 
 def _kernel_shares(fn, top: int = 12) -> List[Tuple[str, float, int]]:
@@ -111,19 +147,20 @@ def measure(cfg, s: Dict[str, int], steps: int, warmup: int, shares: bool) -> Di
     return out
 
 
-def run(steps: int, warmup: int, sizes: List[str], shares: bool) -> Dict[str, Any]:
+def run(design: str, steps: int, warmup: int, names: List[str], shares: bool) -> Dict[str, Any]:
     from ..ops import load_extension
     load_extension()
-    res: Dict[str, Any] = {"metric": "prefill and decode tokens/s, Gebelorn beside the closest Yv model", "dtype": "bf16",
-                           "data": "synthetic uniform-random token ids, random-init weights", "steps": steps, "warmup": warmup,
-                           "time": time.strftime("%Y-%m-%dT%H:%M:%SZ", time.gmtime()), "sizes": {}}
+    sizes, config, closest = DESIGNS[design]
+    res: Dict[str, Any] = {"metric": f"prefill and decode tokens/s, {design.capitalize()} beside the closest Yv model",
+                           "dtype": "bf16", "data": "synthetic uniform-random token ids, random-init weights", "steps": steps,
+                           "warmup": warmup, "time": time.strftime("%Y-%m-%dT%H:%M:%SZ", time.gmtime()), "sizes": {}}
     with torch.no_grad():
-        for name in sizes:
-            s = SIZES[name]
-            res["sizes"][name] = {"shape": s, "gebelorn": measure(design_config(s), s, steps, warmup, shares),
-                                  "closest_yv": measure(closest_config(s), s, steps, warmup, shares)}
+        for name in names or list(sizes):
+            s = sizes[name]
+            res["sizes"][name] = {"shape": s, design: measure(config(s), s, steps, warmup, shares),
+                                  "closest_yv": measure(closest(s), s, steps, warmup, shares)}
     return res
 
 
-def main(steps: int, warmup: int, sizes: str = "", shares: bool = False) -> None:
-    print(json.dumps(run(steps, warmup, [x for x in sizes.split(",") if x] or list(SIZES), shares)))
+def main(design: str, steps: int, warmup: int, sizes: str = "", shares: bool = False) -> None:
+    print(json.dumps(run(design, steps, warmup, [x for x in sizes.split(",") if x], shares)))
