@@ -208,13 +208,6 @@ class YvPagedLayeredCache(YvPagedKVCache):
         return sum(t.numel() * t.element_size() for t in self.k + self.v if t is not None)
 
 
-class YvPagedLatentCache(YvPagedLayeredCache):
-    """Pages of latent rows: layer i stores ``row_sizes[i]`` numbers per token, ``[num_blocks, block_size, row]``."""
-
-    def __init__(self, row_sizes: List[int], cfg: YvCacheConfig, device: torch.device, reach: Optional[int] = None):
-        super().__init__([{"row": r} for r in row_sizes], cfg, device, reach)
-
-
 def cache_for_model(cfg, device: torch.device, num_blocks: int, block_size: Optional[int] = None, tp_size: int = 1,
                     n_layer: Optional[int] = None, dtype: torch.dtype = torch.bfloat16) -> YvPagedKVCache:
     cc = YvCacheConfig(block_size=block_size or cfg.kv_cache_block_size, num_blocks=num_blocks, dtype=dtype)

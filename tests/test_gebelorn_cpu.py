@@ -10,7 +10,7 @@ import torch
 import gebelorn_cases as cases
 import gebelorn_oracle as oracle
 from pisceslx_b200 import YvConfig
-from pisceslx_b200.models.cache import RELEASED, YvCacheConfig, YvPagedLatentCache
+from pisceslx_b200.models.cache import RELEASED, YvCacheConfig, YvPagedLayeredCache
 from pisceslx_b200.models.latent_attention import rotary_for
 from pisceslx_b200.ops import latent as L
 
@@ -167,7 +167,7 @@ def test_pages_behind_every_window_are_given_back_and_used_again(mixed):
 
 
 def test_cache_rows_state_round_trip_and_fork():
-    c = YvPagedLatentCache([6, 10], YvCacheConfig(block_size=4, num_blocks=8, dtype=torch.float32), torch.device("cpu"), reach=5)
+    c = YvPagedLayeredCache([{"row": 6}, {"row": 10}], YvCacheConfig(block_size=4, num_blocks=8, dtype=torch.float32), torch.device("cpu"), reach=5)
     c.add_sequence(1)
     slots = c.append_slots(1, 12)
     assert list(c.slots(1, 0, 12)) == slots
@@ -180,7 +180,7 @@ def test_cache_rows_state_round_trip_and_fork():
     c.free_sequence(1)
     assert c.alloc.available() == 8 - 4
     st = c.state()
-    d = YvPagedLatentCache([6, 10], c.cfg, c.device, reach=5)
+    d = YvPagedLayeredCache([{"row": 6}, {"row": 10}], c.cfg, c.device, reach=5)
     d.load_state(st)
     assert d.tables == c.tables and d.alloc.available() == 4 and d.rows(1).view(-1, 10)[slots[9], 0] == 3.0
     d.free_sequence(2)
