@@ -104,7 +104,7 @@ def test_product_onto_the_stream(M, N, K, dtype):
 # ---- prep ------------------------------------------------------------------------------------------------------------
 @pytest.mark.parametrize("dtype", DTYPES)
 @pytest.mark.parametrize("heads,kv,dim,vdim,rot,unit,temp,bias", [
-    (6, 2, 64, 64, 32, False, None, True), (4, 4, 128, 128, 0, True, (0.3, 5), False), (5, 1, 24, 104, 16, True, (0.2, 1), True),
+    (9, 3, 64, 56, 48, False, None, True), (4, 4, 128, 128, 0, True, (0.3, 5), False), (5, 1, 24, 104, 16, True, (0.2, 1), True),
     (3, 3, 10, 9, 6, True, (0.4, 64), True), (2, 1, 200, 16, 128, True, None, False), (2, 2, 16, 8, 8, False, None, True),
     (8, 2, 128, 64, 128, True, (1.0, 7), True)])
 def test_prep(heads, kv, dim, vdim, rot, unit, temp, bias, dtype):
@@ -180,7 +180,7 @@ def _want(q, ks, vs, nq, heads, scale, sink, gate):
 
 
 SHAPES = [  # heads, kv_heads, dim, vdim, sink, gate
-    (4, 2, 64, 64, True, "element"), (8, 1, 128, 128, False, "head"), (3, 3, 24, 40, True, "head"), (6, 2, 72, 16, True, None),
+    (6, 3, 64, 56, True, "element"), (8, 1, 128, 128, False, "head"), (3, 3, 24, 40, True, "head"), (6, 2, 72, 16, True, None),
     (20, 1, 48, 128, False, "element"), (5, 5, 16, 8, False, None), (34, 2, 128, 64, True, "element")]
 
 
